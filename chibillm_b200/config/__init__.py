@@ -1,9 +1,9 @@
 """Configuration: typed reading of config.json and the architecture registry."""
 from .base import ConfigError, KeyReader, read_config_json
-from .spec import (AdapterSpec, AttentionSpec, DeltaRuleSpec, DenseMLPSpec, FeedForwardSpec, GatedMLPSpec,
-                   GatedRecurrenceSpec, LatentAttentionSpec, LayerSpec, MixerSpec, ModelSpec, NormSpec, PositionSpec,
-                   ParallelMixersSpec, RoutedExpertsSpec, RunStep, ShortConvSpec, StateSpaceSpec, TableExpertsSpec,
-                   TokenInputSpec)
+from .spec import (AdapterSpec, AttentionSpec, ChannelDeltaSpec, DeltaRuleSpec, DenseMLPSpec, FeedForwardSpec,
+                   GatedMLPSpec, GatedRecurrenceSpec, LatentAttentionSpec, LayerSpec, LinearAttentionSpec, MixerSpec,
+                   ModelSpec, NormSpec, PositionSpec, ParallelMixersSpec, RoutedExpertsSpec, RunStep, ShortConvSpec,
+                   StateSpaceSpec, TableExpertsSpec, TokenInputSpec)
 from .registry import (Architecture, find_architecture, load_config, register_architecture,
                        registered_architectures, unregister_architecture)
 from .qwen3 import ARCHITECTURE as QWEN3_ARCHITECTURE, MODEL_TYPE as QWEN3_MODEL_TYPE, Qwen3Config
@@ -23,6 +23,10 @@ register_architecture(PITUDRA_ARCHITECTURE, PitudraConfig.from_dict, PitudraConf
 from .dogetar import ARCHITECTURE as DOGETAR_ARCHITECTURE, DogetarConfig
 
 register_architecture(DOGETAR_ARCHITECTURE, DogetarConfig.from_dict, DogetarConfig.model_spec, replace=True)
+from .pafivik import ARCHITECTURE as PAFIVIK_ARCHITECTURE, SHAPES_KEY as _PAFIVIK_SHAPES, PafivikConfig
+
+register_architecture(PAFIVIK_ARCHITECTURE, PafivikConfig.from_dict, PafivikConfig.model_spec, replace=True,
+                      shapes_key=_PAFIVIK_SHAPES)
 
 __all__ = [
     "ConfigError", "KeyReader", "read_config_json",
@@ -30,6 +34,7 @@ __all__ = [
     "NormSpec", "PositionSpec", "RunStep", "DeltaRuleSpec", "DenseMLPSpec", "ShortConvSpec", "GitipelConfig",
     "TableExpertsSpec", "TokenInputSpec", "FokuraxConfig", "GatedRecurrenceSpec", "LatentAttentionSpec",
     "RoutedExpertsSpec", "PitudraConfig", "StateSpaceSpec", "ParallelMixersSpec", "DogetarConfig",
+    "ChannelDeltaSpec", "LinearAttentionSpec", "PafivikConfig",
     "Architecture", "find_architecture", "load_config", "register_architecture",
     "registered_architectures", "unregister_architecture", "Qwen3Config",
 ]

@@ -52,6 +52,10 @@ class PositionSpec:
     ``factor`` according to their wavelength l = 2 pi / f.  l < original / high keeps f;
     l > original / low gives f / factor; between the two, with
     s = (original / l - low) / (high - low), the frequency is (1 - s) * f / factor + s * f.
+
+    ``interleaved``: features 2i and 2i + 1 form a pair, not i and i + ``rotary_dim`` / 2.  (Scores do
+    not change when q and k are put in another order of features, so a mixer binds its q and k rows in
+    the order that makes the split-half rotation of its kernels this one.)
     """
 
     kind: str
@@ -64,6 +68,7 @@ class PositionSpec:
     slow_turns: float = 0.0
     amplitude_slope: float = 0.0
     wavelength_bands: Optional[Tuple[float, float, float, float]] = None
+    interleaved: bool = False
 
 
 @dataclass(frozen=True)
@@ -266,6 +271,57 @@ class DeltaRuleSpec(MixerSpec):
 
 
 @dataclass(frozen=True)
+class ChannelDeltaSpec(MixerSpec):
+    """The gated delta rule with a decay per head and key channel.  q and k have ``num_kv_heads``
+    heads of ``head_dim`` channels, v ``num_heads`` of ``value_dim``; head h reads q/k head
+    floor(h / (num_heads / num_kv_heads)).  q, k and v (roles "q_proj", "k_proj", "v_proj") pass a
+    causal convolution per channel (``conv_taps`` taps, roles "q_conv", "k_conv", "v_conv"
+    [channels, taps] with the current token's tap last, no bias) and silu; q and k become unit vectors
+    per head, x / sqrt(sum(x^2) + ``key_eps``), and q is multiplied by head_dim^(-1/2).  With
+    b = sigmoid(Wb x) per head (role "b_proj") and, per head and channel,
+    g = exp(-exp(A_log[h]) * softplus(W2 (W1 x) + dt_bias)) (roles "a_log" [num_heads], "decay_in"
+    [``decay_rank``, hidden], "decay_out" [num_heads * head_dim, decay_rank], "dt_bias"):
+
+        S <- diag(g) S,   u = b (v - S^T k),   S <- S + k u^T,   o = S^T q
+
+    (S is head_dim by value_dim, 32-bit, zero at a sequence's start; part of a request's state with the
+    convolutions' last taps - 1 inputs.)  Each head's o is divided by its root mean square
+    (``norm_eps`` inside the root), multiplied by a weight that the heads share (role "out_norm"
+    [value_dim]) and by sigmoid(G2 (G1 x)) (roles "gate_in" [``gate_rank``, hidden], "gate_out"), then
+    projected (role "o_proj")."""
+
+    hidden_size: int = 0
+    num_heads: int = 0
+    num_kv_heads: int = 0
+    head_dim: int = 0
+    value_dim: int = 0
+    conv_taps: int = 1
+    decay_rank: int = 0
+    gate_rank: int = 0
+    key_eps: float = 0.0
+    norm_eps: float = 0.0
+
+
+@dataclass(frozen=True)
+class LinearAttentionSpec(MixerSpec):
+    """Linear attention with a constant decay per head (``decay``, one number each): with
+    q, k = act(Wq x), act(Wk x) (heads of ``head_dim``) and v = act(Wv x) (heads of ``value_dim``),
+    act = silu,
+
+        S <- decay[h] S + k v^T,   o = S^T q       (32-bit, zero at a sequence's start)
+
+    The concatenated heads are divided by their common root mean square (``norm_eps`` inside the root),
+    multiplied by a weight (role "out_norm") and by sigmoid(Wg x) (role "g_proj"), then projected."""
+
+    hidden_size: int = 0
+    num_heads: int = 0
+    head_dim: int = 0
+    value_dim: int = 0
+    decay: Tuple[float, ...] = ()
+    norm_eps: float = 0.0
+
+
+@dataclass(frozen=True)
 class ShortConvSpec:
     """A causal convolution over time on each channel, added to its input:
     y_t = x_t + sum_j w[:, j] * x_(t - taps + 1 + j), zeros before the sequence's
@@ -332,7 +388,11 @@ class RoutedExpertsSpec(FeedForwardSpec):
     choice score, and only outputs of the ``group_keep`` best groups can be chosen.  The last
     ``identity_experts`` outputs name experts without tensors that return their input.
     ``shared_size`` > 0: one more gated expert of that inner size (roles "shared_gate",
-    "shared_up", "shared_down") runs for every token with weight one."""
+    "shared_up", "shared_down") runs for every token with weight one.
+    ``scores`` "sigmoid": s = sigmoid(z), the outputs with the largest s are chosen and s, not
+    renormalised, is the weight.  ``weight_on_input``: the weight multiplies a gated expert's input
+    instead of its output, expert(w * x).  ``shared_output_gate``: the shared expert's output is multiplied
+    by sigmoid(Wsg x), one number per token (role "shared_output_gate" [1, hidden])."""
 
     hidden_size: int = 0
     intermediate_size: int = 0
@@ -347,6 +407,8 @@ class RoutedExpertsSpec(FeedForwardSpec):
     identity_experts: int = 0
     weight_scale: float = 1.0
     shared_size: int = 0
+    weight_on_input: bool = False
+    shared_output_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -371,11 +433,15 @@ class TokenInputSpec:
 @dataclass(frozen=True)
 class DenseMLPSpec(FeedForwardSpec):
     """Dense feed-forward without a gate: down(act(up(x))).  ``activation``:
-    "gelu" (exact, with erf), "gelu_tanh", "silu" or "relu"."""
+    "gelu" (exact, with erf), "gelu_tanh", "silu" or "relu"; or "xielu" with two learned numbers p, q
+    (role "activation" [2]): z > 0 gives softplus(p) z^2 + z / 2, z <= 0 gives
+    (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2.  ``biases`` (with "xielu"): both products add a
+    vector (roles "up_bias", "down_bias")."""
 
     hidden_size: int = 0
     intermediate_size: int = 0
     activation: str = "gelu"
+    biases: bool = False
 
 
 @dataclass(frozen=True)
@@ -410,6 +476,14 @@ class LayerSpec:
     # arrangement "prenorm": the mixer's and the feed-forward's results are multiplied feature by feature
     # by a learned vector each (roles "mixer_scale", "feed_forward_scale") before they join the residual
     layer_scale: bool = False
+    # arrangement "prenorm": norms on the sublayers' results too (roles "mixer_out_norm",
+    # "feed_forward_out_norm"): x += residual_scale * scale * norm(mixer(norm(x))), and the feed-forward alike
+    mixer_out_norm: Optional[NormSpec] = None
+    feed_forward_out_norm: Optional[NormSpec] = None
+    # arrangement "prenorm": with X_0 the embedding output and X_(n) the result of the n-th layer run, what
+    # this block (the ``depth_average``-th run, from 1) hands on is the sum over j = 0 .. depth_average of
+    # w[j] * X_j (role "depth_weights" [depth_average + 1]).  None: off.
+    depth_average: Optional[int] = None
 
     def names(self) -> dict:
         return dict(self.weight_names)

@@ -41,6 +41,8 @@ struct ExpertTileParams {
     void* out;
     long long out_stride;
     int kind;                  // activation of the gate
+    const float* row_weight;   // [pairs] or null: gated sums of pair p's row are multiplied by row_weight[p] first
+    const int* pair_of_row;    // [pairs]
     int* error;
 };
 
@@ -124,6 +126,7 @@ expert_rows_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
         const bool ok = mbar_wait(tmem_full_bar, 0, p.error, 33);
         tcgen05_fence_after();
         const bool write = ok && r < row_end;
+        const float wr = (MODE == 1 && write && p.row_weight) ? p.row_weight[p.pair_of_row[r]] : 1.f;
 #pragma unroll 1
         for (int c0 = 0; c0 < XT_N; c0 += 32) {
             uint32_t v[32];
@@ -163,8 +166,8 @@ expert_rows_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_co
 #pragma unroll
                 for (int j = 0; j < 8; ++j)
                     h[j] = __floats2bfloat162_rn(
-                        activate(__uint_as_float(v[2 * j]), p.kind) * __uint_as_float(v[16 + 2 * j]),
-                        activate(__uint_as_float(v[2 * j + 1]), p.kind) * __uint_as_float(v[16 + 2 * j + 1]));
+                        activate(wr * __uint_as_float(v[2 * j]), p.kind) * (wr * __uint_as_float(v[16 + 2 * j])),
+                        activate(wr * __uint_as_float(v[2 * j + 1]), p.kind) * (wr * __uint_as_float(v[16 + 2 * j + 1])));
                 if (p.out_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0) {
                     reinterpret_cast<uint4*>(dst)[0] = reinterpret_cast<uint4*>(h)[0];
                     reinterpret_cast<uint4*>(dst)[1] = reinterpret_cast<uint4*>(h)[1];
@@ -206,14 +209,14 @@ using namespace chibi;
 // One product of the routed rows on tcgen05.  a: [pairs, K] bfloat16, contiguous, sorted by expert;
 // w: [experts, rows_w, K] bfloat16, contiguous (gated: rows_w = 2 F, interleaved in blocks of 16);
 // route: as route_by_table lays it out for tiles of 128 rows.  out: gated == 1: bfloat16 [pairs, F]
-// with out_stride; gated == 2: bfloat16 [pairs, rows_w], act(sum); else float [pairs, rows_w].  CHIBI_ERR_UNSUPPORTED for sizes it does not take.
+// with out_stride (row_weight [pairs], may be null: see ExpertTileParams); gated == 2: bfloat16 [pairs, rows_w], act(sum); else float [pairs, rows_w].  CHIBI_ERR_UNSUPPORTED for sizes it does not take.
 CHIBI_API int chibi_expert_rows_tc(const void* a, const void* w, void* out, long long out_stride, const int* route,
-                                   long long pairs, int experts, int rows_w, int K, int gated, int kind, int* error,
-                                   cudaStream_t stream)
+                                   long long pairs, int experts, int rows_w, int K, int gated, int kind,
+                                   const float* row_weight, int* error, cudaStream_t stream)
 {
     if (pairs <= 0)
         return CHIBI_OK;
-    if (!a || !w || !out || !route || experts <= 0 || rows_w <= 0 || K <= 0)
+    if (!a || !w || !out || !route || experts <= 0 || rows_w <= 0 || K <= 0 || (row_weight && gated != 1))
         return CHIBI_ERR_ARGUMENT;
     if (K % XT_K != 0 || (gated == 1 && rows_w % 32 != 0) || (reinterpret_cast<uintptr_t>(a) & 15)
         || (reinterpret_cast<uintptr_t>(w) & 15) || pairs > 2147483647LL - XT_M
@@ -234,6 +237,8 @@ CHIBI_API int chibi_expert_rows_tc(const void* a, const void* w, void* out, long
     p.out = out;
     p.out_stride = out_stride;
     p.kind = kind;
+    p.row_weight = row_weight;
+    p.pair_of_row = route + experts + 1;
     p.error = error;
     const dim3 grid((unsigned)((rows_w + XT_N - 1) / XT_N), (unsigned)max_tiles);
     static bool configured = false;

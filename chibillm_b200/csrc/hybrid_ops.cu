@@ -11,7 +11,7 @@
 // * state_space_scan: S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x per head over a step's tokens, from the
 //   request's state to the state it leaves; gated_group_rms: y silu(z) normalised in equal parts;
 // * clamped_swish_gate: min(g, L) sigmoid(s min(g, L)) (clamp(u, -L, L) + 1);
-// * router_choose: softmax over all router outputs, choice by score + correction among the best groups,
+// * router_choose: softmax over all router outputs (or a sigmoid of each), choice by score + correction among the best groups,
 //   weights without the correction; identity_rows: the rows of the experts that return their input;
 // * scaled_add_norm: residual += vec * delta and the next norm's output; add_weighted: acc += a A + b B.
 //
@@ -495,7 +495,7 @@ __global__ void clamped_swish_gate_wide_kernel(const __nv_bfloat16* __restrict__
 __global__ void __launch_bounds__(128)
 router_choose_kernel(const float* __restrict__ logits, long long stride, const float* __restrict__ correction,
                      int* __restrict__ chosen, float* __restrict__ share, long long tokens, int n, int top,
-                     int group_count, int group_keep, float scale, int last_choice)
+                     int group_count, int group_keep, float scale, int last_choice, int sigmoid)
 {
     pdl_enter();
     extern __shared__ float smem[];
@@ -506,18 +506,24 @@ router_choose_kernel(const float* __restrict__ logits, long long stride, const f
     float* score = smem + (size_t)warp * 2 * n;
     float* choice = score + n;
     const float* z = logits + (size_t)t * stride;
-    float m = -INFINITY;
-    for (int i = lane; i < n; i += 32)
-        m = fmaxf(m, z[i]);
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int i = lane; i < n; i += 32) {
-        const float p = expf(z[i] - m);
-        score[i] = p;
-        sum += p;
+    float inv = 1.f;
+    if (sigmoid) {
+        for (int i = lane; i < n; i += 32)
+            score[i] = sigmoid_f(z[i]);
+    } else {
+        float m = -INFINITY;
+        for (int i = lane; i < n; i += 32)
+            m = fmaxf(m, z[i]);
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int i = lane; i < n; i += 32) {
+            const float p = expf(z[i] - m);
+            score[i] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        inv = 1.f / sum;
     }
-    sum = warp_sum(sum);
-    const float inv = 1.f / sum;
     for (int i = lane; i < n; i += 32) {
         score[i] *= inv;
         choice[i] = score[i] + (correction ? correction[i] : 0.f);
@@ -823,7 +829,7 @@ CHIBI_API int chibi_clamped_swish_gate(const void* gate_up, int x_type, long lon
 
 CHIBI_API int chibi_router_choose(const float* logits, long long stride, const float* correction, int* chosen,
                                   float* share, long long tokens, int n, int top, int group_count, int group_keep,
-                                  float scale, int last_choice, cudaStream_t stream)
+                                  float scale, int last_choice, int sigmoid, cudaStream_t stream)
 {
     if (tokens <= 0)
         return CHIBI_OK;
@@ -838,7 +844,7 @@ CHIBI_API int chibi_router_choose(const float* logits, long long stride, const f
         return CHIBI_ERR_UNSUPPORTED;
     const size_t smem = (size_t)warps * 2 * n * sizeof(float);
     launch(router_choose_kernel, dim3((unsigned)blocks), dim3(warps * 32), smem, stream, logits, stride, correction,
-           chosen, share, tokens, n, top, group_count, group_keep, scale, last_choice);
+           chosen, share, tokens, n, top, group_count, group_keep, scale, last_choice, sigmoid);
     return launch_status();
 }
 

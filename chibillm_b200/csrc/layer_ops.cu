@@ -241,6 +241,7 @@ route_by_table_kernel(const int* __restrict__ tokens, const int* __restrict__ ta
 // Tiles of EG_M rows of one expert times 64 columns; 256 threads, a thread owns 4 x 4 sums.
 // out[r, n] = sum_k a[row(r), k] * w[expert][n, k]; GATED: w[expert] holds 2 N rows (gate rows,
 // then up rows) and out[r, n] = act(gate sum) * (up sum); not GATED with kind >= 0: out = act(sum).
+// GATED with row_weight: both sums are first multiplied by row_weight[pair_of_row[r]] (a weight on the row's input).
 // row(r) = a_index[r] / a_div when
 // a_index is given (the rows of the tokens' array that the sorted pairs point at), else r.
 // The K range is walked in order, so a row's sums do not depend on what shares its tile.
@@ -251,7 +252,8 @@ __global__ void __launch_bounds__(256)
 expert_rows_gemm_kernel(const TA* __restrict__ a, long long a_stride, const int* __restrict__ a_index, int a_div,
                         const TW* __restrict__ w, long long w_expert_stride, TO* __restrict__ out,
                         long long out_stride, const int* __restrict__ offsets, const int* __restrict__ tile_expert,
-                        const int* __restrict__ tile_row0, int N, int K, int kind, int interleaved)
+                        const int* __restrict__ tile_row0, int N, int K, int kind, int interleaved,
+                        const float* __restrict__ row_weight, const int* __restrict__ pair_of_row)
 {
     pdl_enter();
     const int expert = tile_expert[blockIdx.y];
@@ -319,6 +321,7 @@ expert_rows_gemm_kernel(const TA* __restrict__ a, long long a_stride, const int*
         const int r = row0 + ty * 4 + i;
         if (r >= row_end)
             continue;
+        const float wr = (GATED && row_weight) ? row_weight[pair_of_row[r]] : 1.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
@@ -326,7 +329,7 @@ expert_rows_gemm_kernel(const TA* __restrict__ a, long long a_stride, const int*
                 continue;
             float v = acc[0][i][j];
             if (GATED)
-                v = activate(v, kind) * acc[GATED ? 1 : 0][i][j];
+                v = activate(wr * v, kind) * (wr * acc[GATED ? 1 : 0][i][j]);
             else if (kind >= 0)
                 v = activate(v, kind);
             out[(size_t)r * out_stride + n] = from_f32<TO>(v);
@@ -375,7 +378,8 @@ __global__ void __launch_bounds__(256, 2)
 expert_rows_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_stride, const int* __restrict__ a_index,
                        int a_div, const __nv_bfloat16* __restrict__ w, long long w_expert_stride, void* __restrict__ out,
                        long long out_stride, const int* __restrict__ offsets, const int* __restrict__ tile_expert,
-                       const int* __restrict__ tile_row0, int N, int K, int kind)
+                       const int* __restrict__ tile_row0, int N, int K, int kind, const float* __restrict__ row_weight,
+                       const int* __restrict__ pair_of_row)
 {
     pdl_enter();
     const int expert = tile_expert[blockIdx.y];
@@ -488,14 +492,15 @@ expert_rows_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_stride, 
             } else if (MODE == 1) {
                 __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(out) + (size_t)r * out_stride;
                 const int base = (n0 + warp_n * 32) / 2;
+                const float wr = row_weight ? row_weight[pair_of_row[r]] : 1.f;
 #pragma unroll
                 for (int ni = 0; ni < 2; ++ni)
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
                         const int col = base + ni * 8 + (lane & 3) * 2 + e;
                         if (col < N / 2)
-                            orow[col] = __float2bfloat16_rn(activate(acc[mi][ni][half * 2 + e], kind)
-                                                            * acc[mi][ni + 2][half * 2 + e]);
+                            orow[col] = __float2bfloat16_rn(activate(wr * acc[mi][ni][half * 2 + e], kind)
+                                                            * (wr * acc[mi][ni + 2][half * 2 + e]));
                     }
             } else {
                 float* orow = static_cast<float*>(out) + (size_t)r * out_stride;
@@ -513,10 +518,13 @@ expert_rows_mma_kernel(const __nv_bfloat16* __restrict__ a, long long a_stride, 
 }
 
 // acc[t, c] += weight * sum over the token's choices (in their order) of y[row_of_pair[t * top + s], c],
-// each times pair_weight[t * top + s] where that is given
+// each times pair_weight[t * top + s] where that is given; with `base` (the sum of `splits` arrays [tokens, n])
+// plus sigmoid(base_gate[t]) * base; `overwrite`: acc is written, not added to
 __global__ void combine_experts_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair,
                                        float* __restrict__ acc, long long acc_stride, long long tokens, int n, int top,
-                                       float weight, const float* __restrict__ pair_weight)
+                                       float weight, const float* __restrict__ pair_weight,
+                                       const float* __restrict__ base, int splits, const float* __restrict__ base_gate,
+                                       long long gate_stride, int overwrite)
 {
     pdl_enter();
     const long long total = tokens * n;
@@ -529,7 +537,51 @@ __global__ void combine_experts_kernel(const float* __restrict__ y, const int* _
             const float v = y[(size_t)row_of_pair[t * top + k] * n + c];
             s = pair_weight ? fmaf(pair_weight[t * top + k], v, s) : s + v;
         }
-        acc[t * acc_stride + c] += weight * s;
+        float v = overwrite ? 0.f : acc[t * acc_stride + c];
+        if (base) {
+            float b = 0.f;
+            for (int k = 0; k < splits; ++k)
+                b += base[(size_t)k * total + i];
+            v = fmaf(b, 1.f / (1.f + expf(-base_gate[t * gate_stride])), v);
+        }
+        acc[t * acc_stride + c] = v + weight * s;
+    }
+}
+
+// The same, four columns (16 bytes of every array) a thread; n and acc_stride are multiples of 4.
+__global__ void combine_experts_wide_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair,
+                                            float* __restrict__ acc, long long acc_stride, long long tokens, int n, int top,
+                                            float weight, const float* __restrict__ pair_weight,
+                                            const float* __restrict__ base, int splits,
+                                            const float* __restrict__ base_gate, long long gate_stride, int overwrite)
+{
+    pdl_enter();
+    const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+    if (c >= n)
+        return;
+    const size_t plane = (size_t)tokens * n;
+    for (long long t = blockIdx.y; t < tokens; t += gridDim.y) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < top; ++k) {
+            const float4 v = *reinterpret_cast<const float4*>(y + (size_t)row_of_pair[t * top + k] * n + c);
+            const float w = pair_weight ? weight * pair_weight[t * top + k] : weight;
+            s.x = fmaf(w, v.x, s.x), s.y = fmaf(w, v.y, s.y), s.z = fmaf(w, v.z, s.z), s.w = fmaf(w, v.w, s.w);
+        }
+        float* dst = acc + t * acc_stride + c;
+        if (!overwrite) {
+            const float4 v = *reinterpret_cast<const float4*>(dst);
+            s.x += v.x, s.y += v.y, s.z += v.z, s.w += v.w;
+        }
+        if (base) {
+            float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int k = 0; k < splits; ++k) {
+                const float4 v = *reinterpret_cast<const float4*>(base + (size_t)k * plane + (size_t)t * n + c);
+                b.x += v.x, b.y += v.y, b.z += v.z, b.w += v.w;
+            }
+            const float g = 1.f / (1.f + expf(-base_gate[t * gate_stride]));
+            s.x = fmaf(g, b.x, s.x), s.y = fmaf(g, b.y, s.y), s.z = fmaf(g, b.z, s.z), s.w = fmaf(g, b.w, s.w);
+        }
+        *reinterpret_cast<float4*>(dst) = s;
     }
 }
 
@@ -776,14 +828,16 @@ CHIBI_API int chibi_route_by_table_open(const int* tokens, const int* table, int
 // tile_rows is what the route was made with: 64 runs the plain kernel (any types and sizes; with
 // interleaved != 0 a gated matrix holds blocks of 16 gate rows and their 16 up rows), 128 the
 // tensor-core kernel (bfloat16, K a multiple of 32, gated matrices interleaved, N a multiple of 16).
+// row_weight [pairs] (may be null; gated 1 only): the sums of pair p's row are multiplied by row_weight[p] before
+// they are activated.
 CHIBI_API int chibi_expert_rows_gemm(const void* a, int a_type, long long a_stride, int gather, int top, const void* w,
                                      int w_type, void* out, long long out_stride, const int* route, long long pairs,
                                      int experts, int N, int K, int gated, int kind, int tile_rows, int interleaved,
-                                     cudaStream_t stream)
+                                     const float* row_weight, cudaStream_t stream)
 {
     if (pairs <= 0)
         return CHIBI_OK;
-    if (!a || !w || !out || !route || N <= 0 || K <= 0 || experts <= 0 || top <= 0
+    if (!a || !w || !out || !route || N <= 0 || K <= 0 || experts <= 0 || top <= 0 || (row_weight && gated != 1)
         || (tile_rows != EG_M && tile_rows != TG_M))
         return CHIBI_ERR_ARGUMENT;
     const int max_tiles = (int)((pairs + tile_rows - 1) / tile_rows) + experts;
@@ -807,7 +861,7 @@ CHIBI_API int chibi_expert_rows_gemm(const void* a, int a_type, long long a_stri
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch(kernel, tgrid, dim3(256), smem, stream, (const __nv_bfloat16*)a, a_stride,
                gather ? pair_of_row : (const int*)nullptr, top, (const __nv_bfloat16*)w, w_stride, out, out_stride,
-               offsets, tile_expert, tile_row0, rows_of_w, K, kind);
+               offsets, tile_expert, tile_row0, rows_of_w, K, kind, row_weight, pair_of_row);
         return launch_status();
     }
     const dim3 grid((unsigned)((N + EG_N - 1) / EG_N), (unsigned)max_tiles);
@@ -815,16 +869,42 @@ CHIBI_API int chibi_expert_rows_gemm(const void* a, int a_type, long long a_stri
         if (gated == 1)
             launch(expert_rows_gemm_kernel<TA, TW, TA, true>, grid, dim3(256), 0, stream, (const TA*)a, a_stride,
                    gather ? pair_of_row : (const int*)nullptr, top, (const TW*)w, w_stride, (TA*)out, out_stride,
-                   offsets, tile_expert, tile_row0, N, K, kind, interleaved);
+                   offsets, tile_expert, tile_row0, N, K, kind, interleaved, row_weight, pair_of_row);
         else if (gated == 2)
             launch(expert_rows_gemm_kernel<TA, TW, TA, false>, grid, dim3(256), 0, stream, (const TA*)a, a_stride,
                    gather ? pair_of_row : (const int*)nullptr, top, (const TW*)w, w_stride, (TA*)out, out_stride,
-                   offsets, tile_expert, tile_row0, N, K, kind, 0);
+                   offsets, tile_expert, tile_row0, N, K, kind, 0, row_weight, pair_of_row);
         else
             launch(expert_rows_gemm_kernel<TA, TW, float, false>, grid, dim3(256), 0, stream, (const TA*)a, a_stride,
                    gather ? pair_of_row : (const int*)nullptr, top, (const TW*)w, w_stride, (float*)out, out_stride,
-                   offsets, tile_expert, tile_row0, N, K, -1, 0);
+                   offsets, tile_expert, tile_row0, N, K, -1, 0, row_weight, pair_of_row);
     }));
+    return launch_status();
+}
+
+// `base` (may be null): [splits, tokens, n], joined as sigmoid(base_gate[t * gate_stride]) * (the splits' sum)
+CHIBI_API int chibi_combine_experts_onto(const float* y, const int* route, float* acc, long long acc_stride,
+                                         long long tokens, int n, int top, int experts, float weight,
+                                         const float* pair_weight, const float* base, int splits,
+                                         const float* base_gate, long long gate_stride, int overwrite,
+                                         cudaStream_t stream)
+{
+    if (tokens <= 0)
+        return CHIBI_OK;
+    if (!y || !route || !acc || n <= 0 || top <= 0 || (base && (!base_gate || splits < 1)))
+        return CHIBI_ERR_ARGUMENT;
+    const int* row_of_pair = route + experts + 1 + tokens * top;
+    const uintptr_t all = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(acc) | reinterpret_cast<uintptr_t>(base);
+    if (n % 4 == 0 && acc_stride % 4 == 0 && (all & 15) == 0) {
+        const int threads = n / 4 < 256 ? (n / 4 + 31) / 32 * 32 : 256;
+        launch(combine_experts_wide_kernel, dim3((unsigned)((n / 4 + threads - 1) / threads),
+                                                 (unsigned)(tokens < 32768 ? tokens : 32768)),
+               dim3(threads), 0, stream, y, row_of_pair, acc, acc_stride, tokens, n, top, weight, pair_weight, base, splits,
+               base_gate, gate_stride, overwrite);
+        return launch_status();
+    }
+    launch(combine_experts_kernel, dim3(blocks_for(tokens * n, 256)), dim3(256), 0, stream, y, row_of_pair, acc,
+           acc_stride, tokens, n, top, weight, pair_weight, base, splits, base_gate, gate_stride, overwrite);
     return launch_status();
 }
 
@@ -832,14 +912,8 @@ CHIBI_API int chibi_combine_experts(const float* y, const int* route, float* acc
                                     long long tokens, int n, int top, int experts, float weight,
                                     const float* pair_weight, cudaStream_t stream)
 {
-    if (tokens <= 0)
-        return CHIBI_OK;
-    if (!y || !route || !acc || n <= 0 || top <= 0)
-        return CHIBI_ERR_ARGUMENT;
-    const int* row_of_pair = route + experts + 1 + tokens * top;
-    launch(combine_experts_kernel, dim3(blocks_for(tokens * n, 256)), dim3(256), 0, stream, y, row_of_pair, acc,
-           acc_stride, tokens, n, top, weight, pair_weight);
-    return launch_status();
+    return chibi_combine_experts_onto(y, route, acc, acc_stride, tokens, n, top, experts, weight, pair_weight, nullptr, 1,
+                                      nullptr, 0, 0, stream);
 }
 
 CHIBI_API int chibi_layer_end(float* residual, const float* delta, float mult, const int* tokens,

@@ -37,6 +37,16 @@ class DecoderModel:
                 raise ValueError(f"run step {i} names stream adapter {step.enter}; the model has "
                                  f"{len(self.stream_adapters)}")
         self._keep_embedding_output = any(a.needs_embedding_output for a in self.stream_adapters)
+        # blocks that hand on a weighted sum over the embedding output and all blocks' results so far
+        self._depth = 0
+        for i, step in enumerate(spec.run_order):
+            earlier = getattr(spec.layers[step.layer], "depth_average", None)
+            if earlier is not None:
+                if earlier != i + 1:
+                    raise ValueError(f"run step {i} averages over {earlier} earlier results; there are {i + 1}")
+                self._depth = i + 1
+        if self._depth not in (0, len(spec.run_order)):
+            raise ValueError("either every run step or none averages over the results so far")
 
     # ---- weights
     def expected_tensors(self, available: Optional[Iterable[str]] = None) -> List[TensorSpec]:
@@ -114,6 +124,11 @@ class DecoderModel:
             kept = ctx.workspace.get("model.embedding_output", (T, hidden), torch.float32)
             k.cast(residual, kept)
             ctx.shared["embedding output"] = kept
+        if self._depth:
+            # X_0, X_1, ...: the embedding output, then every block's result (the last one's is not kept)
+            outputs = ctx.workspace.get("model.layer_outputs", (self._depth, T, hidden), torch.float32)
+            k.cast(residual, outputs[0])
+            ctx.shared["layer outputs"] = outputs
         pending = None      # a last product that a block left to be added to the residual
         for i, step in enumerate(self.spec.run_order):
             if step.enter is not None:

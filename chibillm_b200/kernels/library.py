@@ -59,7 +59,7 @@ _SIGNATURES = {
         "chibi_heads_rotate_append": [P, I, L, P, P, P, I, P, F, P, P, P, P, I, L, I, I, I, I, I, I, I, F, I, I, P, P],
         "chibi_gated_activation": [P, I, L, P, I, P, L, I, I, I, P],
         "chibi_route_by_table": [P, P, I, I, I, L, I, P, P, P],
-        "chibi_expert_rows_gemm": [P, I, L, I, I, P, I, P, L, P, L, I, I, I, I, I, I, I, P],
+        "chibi_expert_rows_gemm": [P, I, L, I, I, P, I, P, L, P, L, I, I, I, I, I, I, I, P, P],
         "chibi_combine_experts": [P, P, P, L, L, I, I, I, F, P, P],
         "chibi_norm_rows": [P, P, P, I, F, F, I, P, P, I, L, I, P],
         "chibi_token_shift": [P, P, P, P, P, P, P, I, L, I, P],
@@ -74,7 +74,7 @@ _SIGNATURES = {
         "chibi_softcap": [P, F, L, P],
         "chibi_zero": [P, L, P],
         "chibi_expert_tile_rows": [],
-        "chibi_expert_rows_tc": [P, P, P, L, P, L, I, I, I, I, I, P, P],
+        "chibi_expert_rows_tc": [P, P, P, L, P, L, I, I, I, I, I, P, P, P],
         "chibi_expert_tile_rows_tensor_cores": [],
         "chibi_attention_generic_shared": [P, I, P, P, I, P, I, P, I, P, P, P, P, P, L, I, I, I, I, I, I, F, I, I, F, P, P,
                                            P, I, P, P],
@@ -88,9 +88,16 @@ _SIGNATURES = {
         "chibi_state_space_scan": [P, I, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P],
         "chibi_gated_group_rms": [P, P, I, L, P, F, P, L, I, I, P],
         "chibi_clamped_swish_gate": [P, I, L, P, L, I, F, F, P],
-        "chibi_router_choose": [P, L, P, P, P, L, I, I, I, I, F, I, P],
+        "chibi_router_choose": [P, L, P, P, P, L, I, I, I, I, F, I, I, P],
         "chibi_identity_rows": [P, I, L, P, P, L, I, I, I, I, P],
         "chibi_scaled_add_norm": [P, P, P, P, I, F, F, P, I, L, I, P],
+        "chibi_combine_experts_onto": [P, P, P, L, L, I, I, I, F, P, P, I, P, L, I, P],
+        "chibi_sublayer_end": [P, P, I, P, P, F, P, P, I, I, P, I, F, F, P, I, L, I, P],
+        "chibi_norm_then_gate": [P, P, I, L, P, F, P, L, I, P],
+        "chibi_bias_xielu": [P, I, I, P, P, I, L, I, F, F, P],
+        "chibi_recurrence_scratch": [L, I, I, I, I, P],
+        "chibi_channel_delta": [P, I, L, P, L, P, L, P, P, P, P, P, L, P, P, L, I, I, I, I, I, I, F, F, I, P],
+        "chibi_decayed_attention": [P, I, L, I, P, P, P, P, L, P, P, L, I, I, I, I, I, I, P],
     },
     "chibi_attention_tc": {
         "chibi_attention_tc_head_dim": [],

@@ -654,8 +654,8 @@ class CudaKernels:
     def linear(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor,
                residual: Optional[torch.Tensor] = None, defer: bool = False) -> Optional[PendingSum]:
         """out[M, N] = x[M, K] @ w[N, K]^T (+ residual, 32-bit, may alias out).
-        With ``defer`` (only together with a residual that aliases out) a split
-        product is left pending -- the caller adds it later -- and is returned."""
+        With ``defer`` (together with a residual that aliases out, or without one) a split
+        product is left pending -- the caller adds it, or takes it for ``out`` -- and is returned."""
         if isinstance(x, ScaledRows):
             if residual is None and self._linear_of_scaled(x, w, out, swiglu=False):
                 return None
@@ -667,6 +667,10 @@ class CudaKernels:
             if self.use_tensor_cores and self.fold_norms and x.shape[0] > self.few_rows_max and x.dtype == torch.bfloat16 \
                     and w.dtype == torch.bfloat16 and residual.dtype == torch.float32:
                 return DeferredProduct(self, x, w)
+        elif defer and residual is None:
+            pending = self.linear_partial(x, w)
+            if pending is not None:
+                return pending
         _need_cuda(x, w, out, residual)
         _rows_contiguous(x, "linear: x")
         _rows_contiguous(w, "linear: w")
@@ -1313,10 +1317,10 @@ class CudaKernels:
             rows = route[E + 1 + 2 * pairs + 2 * max_tiles:E + 1 + 3 * pairs + 2 * max_tiles]
             self.gather_rows(x, rows, sorted_x)
             s1 = self.lib.chibi_expert_rows_tc(_ptr(sorted_x), _ptr(gate_up), _ptr(act), F, _ptr(route), pairs, E,
-                                               2 * F, D, 1, self.ACTIVATIONS[kind], _ptr(self.error), stream)
+                                               2 * F, D, 1, self.ACTIVATIONS[kind], None, _ptr(self.error), stream)
             if s1 == 0:
                 _check(self.lib.chibi_expert_rows_tc(_ptr(act), _ptr(down), _ptr(y), D, _ptr(route), pairs, E, D, F, 0,
-                                                     0, _ptr(self.error), stream), "routed_experts (down, tcgen05)")
+                                                     0, None, _ptr(self.error), stream), "routed_experts (down, tcgen05)")
                 _check(self.lib.chibi_combine_experts(_ptr(y), _ptr(route), _ptr(acc), acc.stride(0), T, D, top, E,
                                                       float(weight), None, stream), "routed_experts (combine)")
                 self.tensor_core_calls += 2
@@ -1325,9 +1329,9 @@ class CudaKernels:
                 _check(s1, "routed_experts (gate | up, tcgen05)")
         _check(self.lib.chibi_expert_rows_gemm(_ptr(x), _code(x), x.stride(0), 1, top, _ptr(gate_up), _code(gate_up),
                                                _ptr(act), F, _ptr(route), pairs, E, F, D, 1, self.ACTIVATIONS[kind],
-                                               tile, flag, stream), "routed_experts (gate | up)")
+                                               tile, flag, None, stream), "routed_experts (gate | up)")
         _check(self.lib.chibi_expert_rows_gemm(_ptr(act), _code(act), F, 0, top, _ptr(down), _code(down), _ptr(y), D,
-                                               _ptr(route), pairs, E, D, F, 0, 0, tile, 0, stream),
+                                               _ptr(route), pairs, E, D, F, 0, 0, tile, 0, None, stream),
                "routed_experts (down)")
         if fast:
             self.tensor_core_calls += 2
@@ -1526,7 +1530,8 @@ class CudaKernels:
     def chosen_experts(self, x: torch.Tensor, chosen: torch.Tensor, share: torch.Tensor, up: torch.Tensor,
                        down: torch.Tensor, acc: torch.Tensor, route: torch.Tensor, act: torch.Tensor, y: torch.Tensor,
                        kind: str, sorted_x: Optional[torch.Tensor] = None, gated: bool = False,
-                       interleaved: bool = False, identity: int = 0) -> None:
+                       interleaved: bool = False, identity: int = 0, weight_on_input: bool = False, base=None,
+                       overwrite: bool = False) -> None:
         """acc[t] += sum over s of share[t, s] * down_e (act(up_e x[t])), e = chosen[t, s]; up
         [E, F, D], down [E, D, F]; scratch as for ``routed_experts``.  The (token, choice)
         pairs are sorted by expert on the device and the two products run over tiles of one
@@ -1535,7 +1540,11 @@ class CudaKernels:
         ``interleave_expert_gate_up`` lays them), and an expert is down(act(gate x) * (up x)).
         ``identity`` n > 0: choice E - 1 names the experts that return their input (times the
         share); the last of the E stacked matrices is a stand-in that is never read, and the
-        bucket of these choices gets no tiles: its rows take the tokens' inputs instead."""
+        bucket of these choices gets no tiles: its rows take the tokens' inputs instead.
+        ``weight_on_input`` (gated): the share multiplies the expert's input, not its output (the first
+        product multiplies its 32-bit sums by it).  ``base`` (b, gate): sigmoid(gate[t]) * b[t] joins the sum, b
+        a float32 array [T, D] or a PendingSum, gate float32 [T, 1].  ``overwrite``: acc holds nothing yet
+        and is written."""
         _need_cuda(x, chosen, share, up, down, acc, route, act, y)
         _rows_contiguous(x, "chosen_experts: x")
         _rows_contiguous(acc, "chosen_experts: acc")
@@ -1554,6 +1563,28 @@ class CudaKernels:
                 or y.shape != (pairs, D) or y.dtype != torch.float32 or not y.is_contiguous()
                 or kind not in self.ACTIVATIONS):
             raise KernelError("chosen_experts: shapes or types")
+        if weight_on_input and (not gated or identity):
+            raise KernelError("chosen_experts: weights on the inputs belong to gated experts, none of them an identity")
+        row_weight, pair_weight = (_ptr(share), None) if weight_on_input else (None, _ptr(share))
+        base_ptr = gate_ptr = None
+        splits, gate_stride = 1, 0
+        if base is not None:
+            b, gate = base
+            if isinstance(b, PendingSum):
+                splits, shape, b = b.splits, (b.M, b.N), b.partial
+            else:
+                shape = tuple(b.shape)
+            _need_cuda(b, gate)
+            if shape != (T, D) or b.dtype != torch.float32 or not b.is_contiguous() or gate.dtype != torch.float32 \
+                    or gate.shape != (T, 1):
+                raise KernelError("chosen_experts: base float32 [T, D] and its gate float32 [T, 1]")
+            base_ptr, gate_ptr, gate_stride = _ptr(b), _ptr(gate), gate.stride(0)
+
+        def combine():
+            _check(self.lib.chibi_combine_experts_onto(
+                _ptr(y), _ptr(route), _ptr(acc), acc.stride(0), T, D, top, E, 1.0, pair_weight, base_ptr, splits, gate_ptr,
+                gate_stride, 1 if overwrite else 0, stream), "chosen_experts (combine)")
+
         stream = self._stream()
         self.launches += 4
         # as ``routed_experts``: bfloat16 experts of sizes that are multiples of 32 run on the tensor cores
@@ -1583,26 +1614,25 @@ class CudaKernels:
             rows = route[E + 1 + 2 * pairs + 2 * max_tiles:E + 1 + 3 * pairs + 2 * max_tiles]
             self.gather_rows(x, rows, sorted_x)
             s1 = self.lib.chibi_expert_rows_tc(_ptr(sorted_x), _ptr(up), _ptr(act), F, _ptr(route), pairs, E, rows_up, D,
-                                               first, code, _ptr(self.error), stream)
+                                               first, code, row_weight, _ptr(self.error), stream)
             if s1 == 0:
                 _check(self.lib.chibi_expert_rows_tc(_ptr(act), _ptr(down), _ptr(y), D, _ptr(route), pairs, E, D, F, 0,
-                                                     0, _ptr(self.error), stream), "chosen_experts (down, tcgen05)")
-                _check(self.lib.chibi_combine_experts(_ptr(y), _ptr(route), _ptr(acc), acc.stride(0), T, D, top, E,
-                                                      1.0, _ptr(share), stream), "chosen_experts (combine)")
+                                                     0, None, _ptr(self.error), stream), "chosen_experts (down, tcgen05)")
+                combine()
                 self.tensor_core_calls += 2
                 return
             if s1 != -2:
                 _check(s1, "chosen_experts (up, tcgen05)")
         _check(self.lib.chibi_expert_rows_gemm(_ptr(x), _code(x), x.stride(0), 1, top, _ptr(up), _code(up), _ptr(act),
-                                               F, _ptr(route), pairs, E, F, D, first, code, tile, flag, stream),
+                                               F, _ptr(route), pairs, E, F, D, first, code, tile, flag, row_weight,
+                                               stream),
                "chosen_experts (up)")
         _check(self.lib.chibi_expert_rows_gemm(_ptr(act), _code(act), F, 0, top, _ptr(down), _code(down), _ptr(y), D,
-                                               _ptr(route), pairs, E, D, F, 0, 0, tile, 0, stream),
+                                               _ptr(route), pairs, E, D, F, 0, 0, tile, 0, None, stream),
                "chosen_experts (down)")
         if fast:
             self.tensor_core_calls += 2
-        _check(self.lib.chibi_combine_experts(_ptr(y), _ptr(route), _ptr(acc), acc.stride(0), T, D, top, E, 1.0,
-                                              _ptr(share), stream), "chosen_experts (combine)")
+        combine()
 
     def layer_end(self, residual: torch.Tensor, delta: Optional[torch.Tensor], mult: float, side=None,
                   y_in: Optional[torch.Tensor] = None, norm=None, copy_out: Optional[torch.Tensor] = None) -> None:
@@ -1851,8 +1881,8 @@ class CudaKernels:
 
     def router_choose(self, logits: torch.Tensor, correction: Optional[torch.Tensor], chosen: torch.Tensor,
                       share: torch.Tensor, group_count: int, group_keep: int, scale: float,
-                      last_choice: Optional[int] = None) -> None:
-        """s = softmax(logits[t]) (float32 [T, n]); choice = s + correction; of ``group_count`` equal
+                      last_choice: Optional[int] = None, sigmoid: bool = False) -> None:
+        """s = softmax(logits[t]) (``sigmoid``: of every logit by itself) (float32 [T, n]); choice = s + correction; of ``group_count`` equal
         groups of neighbours only the ``group_keep`` with the largest best choice stay open;
         chosen[t] (int32 [T, top]) = the open outputs with the largest choice, largest first, ties to
         the lower number; share[t] = s[chosen] * scale.  ``last_choice``: numbers above it are written
@@ -1870,8 +1900,8 @@ class CudaKernels:
         self.launches += 1
         _check(self.lib.chibi_router_choose(_ptr(logits), logits.stride(0), _ptr(correction), _ptr(chosen),
                                             _ptr(share), T, n, top, int(group_count), int(group_keep), float(scale),
-                                            n - 1 if last_choice is None else int(last_choice), self._stream()),
-               "router_choose")
+                                            n - 1 if last_choice is None else int(last_choice),
+                                            1 if sigmoid else 0, self._stream()), "router_choose")
 
     def scaled_add_norm(self, residual: torch.Tensor, delta: torch.Tensor, vec: Optional[torch.Tensor],
                         norm=None) -> None:
@@ -1895,6 +1925,145 @@ class CudaKernels:
                                               _code(w) if w is not None else F32, float(eps), float(offset),
                                               _ptr(out), _code(out) if out is not None else F32, T, n,
                                               self._stream()), "scaled_add_norm")
+
+    # ---- parts of linear_recurrence.cu
+    # steps whose sequences bring at most so many tokens run the recurrences token by token, others in
+    # chunks of 16 tokens
+    RECURRENCE_FEW_TOKENS = 4
+
+    def _recurrence_scratch(self, tokens: int, seqs: int, heads: int, d: int, delta: bool, max_q_len: int):
+        if max_q_len <= self.RECURRENCE_FEW_TOKENS:
+            return None
+        floats = ctypes.c_longlong(0)
+        _check(self.lib.chibi_recurrence_scratch(tokens, seqs, heads, d, 1 if delta else 0, ctypes.addressof(floats)),
+               "recurrence scratch")
+        return self._scratch(floats.value)
+
+    def channel_delta(self, qkv: torch.Tensor, logits: torch.Tensor, beta: torch.Tensor, a_log: torch.Tensor,
+                      dt_bias: torch.Tensor, state: torch.Tensor, o: torch.Tensor, q_start: torch.Tensor,
+                      state_slots: torch.Tensor, heads: int, kv_heads: int, d: int, e: int, key_eps: float,
+                      q_scale: float, max_q_len: int) -> None:
+        """The gated delta rule with a decay per key channel, over the step's tokens of every sequence, from
+        and to ``state`` (float32 [slots, heads, d, e]).  qkv [T, 2 kv_heads d + heads e] holds q | k | v; per
+        head h (q/k head h // (heads / kv_heads)): q and k divided by sqrt(sum of squares + key_eps), q times
+        q_scale; b = sigmoid(beta[t, h]); g = exp(-exp(a_log[h]) softplus(logits[t, h d + c] + dt_bias[h d + c]));
+        S <- diag(g) S; u = b (v - S^T k); S <- S + k u^T; o = S^T q (float32 [T, heads e])."""
+        _need_cuda(qkv, logits, beta, a_log, dt_bias, state, o, q_start, state_slots)
+        for t, what in ((qkv, "qkv"), (logits, "logits"), (beta, "beta")):
+            _rows_contiguous(t, f"channel_delta: {what}")
+        T = qkv.shape[0]
+        if qkv.shape[1] != 2 * kv_heads * d + heads * e or logits.shape != (T, heads * d) or logits.dtype != torch.float32 \
+                or beta.shape != (T, heads) or beta.dtype != qkv.dtype or state.dtype != torch.float32 \
+                or tuple(state.shape[1:]) != (heads, d, e) or not state.is_contiguous() or o.dtype != torch.float32 \
+                or o.shape != (T, heads * e) or not o.is_contiguous():
+            raise KernelError("channel_delta: shapes or types")
+        for t, size in ((a_log, heads), (dt_bias, heads * d)):
+            if t.dtype != torch.float32 or t.numel() != size or not t.is_contiguous():
+                raise KernelError("channel_delta: a_log [heads] and dt_bias [heads d] are contiguous float32")
+        seqs = state_slots.numel()
+        scratch = self._recurrence_scratch(T, seqs, heads, d, True, max_q_len)
+        self.launches += 2 if scratch is not None and d <= 256 else 1
+        _check(self.lib.chibi_channel_delta(
+            _ptr(qkv), _code(qkv), qkv.stride(0), _ptr(logits), logits.stride(0), _ptr(beta), beta.stride(0), _ptr(a_log),
+            _ptr(dt_bias), _ptr(state), _ptr(o), _ptr(scratch), scratch.numel() if scratch is not None else 0,
+            _ptr(q_start), _ptr(state_slots), T, seqs, int(max_q_len), heads, kv_heads, d, e, float(key_eps),
+            float(q_scale), self.RECURRENCE_FEW_TOKENS, self._stream()), "channel_delta")
+
+    def decayed_attention(self, qkv: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, o: torch.Tensor,
+                          q_start: torch.Tensor, state_slots: torch.Tensor, heads: int, d: int, e: int, max_q_len: int,
+                          activate: bool = False) -> None:
+        """Linear attention with a constant decay per head, over the step's tokens of every sequence, from and to
+        ``state`` (float32 [slots, heads, d, e]).  qkv [T, 2 heads d + heads e] holds q | k | v (with
+        ``activate`` before their silu): S <- decay[h] S + k v^T, o = S^T q (float32 [T, heads e])."""
+        _need_cuda(qkv, decay, state, o, q_start, state_slots)
+        _rows_contiguous(qkv, "decayed_attention: qkv")
+        T = qkv.shape[0]
+        if qkv.shape[1] != heads * (2 * d + e) or decay.dtype != torch.float32 or decay.numel() != heads \
+                or state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, d, e) or not state.is_contiguous() \
+                or o.dtype != torch.float32 or o.shape != (T, heads * e) or not o.is_contiguous():
+            raise KernelError("decayed_attention: shapes or types")
+        seqs = state_slots.numel()
+        scratch = self._recurrence_scratch(T, seqs, heads, d, False, max_q_len)
+        self.launches += 2 if scratch is not None and d <= 256 else 1
+        _check(self.lib.chibi_decayed_attention(
+            _ptr(qkv), _code(qkv), qkv.stride(0), 1 if activate else 0, _ptr(decay), _ptr(state), _ptr(o), _ptr(scratch),
+            scratch.numel() if scratch is not None else 0, _ptr(q_start), _ptr(state_slots), T, seqs, int(max_q_len),
+            heads, d, e, self.RECURRENCE_FEW_TOKENS, self._stream()), "decayed_attention")
+
+    # ---- parts of sublayer_ops.cu
+    def norm_then_gate(self, x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float,
+                       out: torch.Tensor) -> None:
+        """out = x / sqrt(mean(x^2 over the row) + eps) * weight * sigmoid(gate); x float32 [T, n], gate of out's type."""
+        _need_cuda(x, gate, weight, out)
+        _rows_contiguous(gate, "norm_then_gate: gate")
+        T, n = x.shape
+        if x.dtype != torch.float32 or not x.is_contiguous() or gate.shape != x.shape or gate.dtype != out.dtype \
+                or weight.dtype != torch.float32 or weight.shape != (n,) or not weight.is_contiguous() \
+                or out.shape != x.shape or not out.is_contiguous():
+            raise KernelError("norm_then_gate: shapes or types")
+        self.launches += 1
+        _check(self.lib.chibi_norm_then_gate(_ptr(x), _ptr(gate), _code(gate), gate.stride(0), _ptr(weight), float(eps),
+                                             _ptr(out), T, n, self._stream()), "norm_then_gate")
+
+    def bias_xielu(self, x, bias: Optional[torch.Tensor], out: torch.Tensor, curve_pos: float, curve_neg: float) -> None:
+        """z = x + bias; out = curve_pos z^2 + z / 2 for z > 0, curve_neg (exp(z) - 1 - z) + z / 2 otherwise;
+        x [T, n] (may be out) or a PendingSum, bias float32 [n]."""
+        splits = 1
+        if isinstance(x, PendingSum):
+            splits, shape, x = x.splits, (x.M, x.N), x.partial
+        else:
+            shape = tuple(x.shape)
+        _need_cuda(x, bias, out)
+        T, n = out.shape
+        if shape != (T, n) or not x.is_contiguous() or not out.is_contiguous() \
+                or (bias is not None and (bias.dtype != torch.float32 or bias.shape != (n,) or not bias.is_contiguous())):
+            raise KernelError("bias_xielu: shapes or types")
+        self.launches += 1
+        _check(self.lib.chibi_bias_xielu(_ptr(x), _code(x), splits, _ptr(bias), _ptr(out), _code(out), T, n,
+                                         float(curve_pos), float(curve_neg), self._stream()), "bias_xielu")
+
+    def sublayer_end(self, residual: torch.Tensor, delta, vec: torch.Tensor, eps: Optional[float],
+                     bias: Optional[torch.Tensor], depth=None, norm=None) -> None:
+        """y = delta + bias (delta float32 [T, n] or a PendingSum); residual += vec * y / sqrt(mean(y^2) + eps)
+        (eps None: vec * y).  ``depth`` (outputs [N, T, n], j, weights [j + 1]): the new residual is kept as
+        outputs[j] (if there is such a place) and replaced by weights[j] * it + the sum of
+        weights[i] * outputs[i] over i < j.  ``norm`` (weight, eps, offset, out): then out = the residual's
+        RMS norm.  One launch."""
+        splits = 1
+        if isinstance(delta, PendingSum):
+            splits, shape, delta = delta.splits, (delta.M, delta.N), delta.partial
+        else:
+            shape = tuple(delta.shape)
+        _need_cuda(residual, delta, vec, bias)
+        T, n = residual.shape
+        if residual.dtype != torch.float32 or not residual.is_contiguous() or shape != (T, n) \
+                or delta.dtype != torch.float32 or not delta.is_contiguous():
+            raise KernelError("sublayer_end: contiguous float32 residual and delta [T, n]")
+        for t in (vec, bias):
+            if t is not None and (t.dtype != torch.float32 or t.shape != (n,) or not t.is_contiguous()):
+                raise KernelError("sublayer_end: vec and bias are contiguous float32 [n]")
+        outputs = weights = None
+        earlier = keep = 0
+        if depth is not None:
+            outputs, earlier, weights = depth
+            _need_cuda(outputs, weights)
+            keep = 1 if earlier < outputs.shape[0] else 0
+            if outputs.dtype != torch.float32 or not outputs.is_contiguous() or tuple(outputs.shape[1:]) != (T, n) \
+                    or not 0 < earlier <= outputs.shape[0] or weights.dtype != torch.float32 \
+                    or weights.shape != (earlier + 1,) or not weights.is_contiguous():
+                raise KernelError("sublayer_end: outputs float32 [N, T, n] and weights [j + 1]")
+        w = out = None
+        n_eps = offset = 0.0
+        if norm is not None:
+            w, n_eps, offset, out = norm
+            _need_cuda(w, out)
+            if w.shape != (n,) or not w.is_contiguous() or out.shape != (T, n) or not out.is_contiguous():
+                raise KernelError("sublayer_end: shapes of the norm")
+        self.launches += 1
+        _check(self.lib.chibi_sublayer_end(
+            _ptr(residual), _ptr(delta), splits, _ptr(bias), _ptr(vec), -1.0 if eps is None else float(eps), _ptr(outputs),
+            _ptr(weights), int(earlier), keep, _ptr(w), _code(w) if w is not None else F32, float(n_eps), float(offset),
+            _ptr(out), _code(out) if out is not None else F32, T, n, self._stream()), "sublayer_end")
 
     def softcap(self, x: torch.Tensor, cap: float) -> None:
         """x = cap * tanh(x / cap), in place (float32)."""

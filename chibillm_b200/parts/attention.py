@@ -43,6 +43,9 @@ head with the shared weight, rotates, writes q and appends k and v (the maps of 
 head are key heads of the cache that share one value head); attention follows, 32-bit
 where maps are to be subtracted; one kernel joins the maps, normalises and gates; then
 the output product.
+
+A rotation of neighbouring features (``PositionSpec.interleaved``) is the kernels' split-half rotation with
+the rows of every q and k head (and their biases and norm weights) put in another order when they are bound.
 """
 from __future__ import annotations
 
@@ -93,6 +96,8 @@ class PagedAttention(Mixer):
         self.value_dim = spec.head_dim if spec.value_dim is None else spec.value_dim
         if spec.tied_values and self.value_dim != spec.head_dim:
             raise ValueError("values tied to the keys have the keys' size")
+        if spec.tied_values and self.position.feature_order() is not None:
+            raise ValueError("values tied to the keys are not combined with a rotation of neighbouring features")
         if spec.unit_norm_eps is not None and spec.qk_norm is not None:
             raise ValueError("a norm of q and k comes either before the rotation (qk_norm) or after it (unit_norm_eps)")
         if self.prepared:
@@ -175,6 +180,15 @@ class PagedAttention(Mixer):
             self.slopes = torch.tensor([2.0 ** (-float(self.spec.distance_slope_bits) * (h + 1) / H)
                                         for h in range(H)], dtype=torch.float32,
                                        device=tensors[self.names["q_proj"]].device)
+        order = self.position.feature_order()
+        if order is not None:
+            # the features of q and k in the order in which the kernels' rotation pairs them
+            tensors = dict(tensors)
+            d = self.spec.head_dim
+            for r in ("q_proj", "k_proj", "q_bias", "k_bias", "q_norm", "k_norm"):
+                t = tensors.get(self.names.get(r))
+                if t is not None:
+                    tensors[self.names[r]] = t.view(-1, d, *t.shape[1:])[:, order.to(t.device)].reshape(t.shape)
         mats = [tensors[self.names[r]] for r in roles]
         if self.maps > 1:
             # Query rows come head by head, a head's maps side by side; a key head of the cache is one map
@@ -204,6 +218,7 @@ class PagedAttention(Mixer):
 
     # ---- cache
     accepts_scaled_rows = True       # x goes to the q | k | v product and nowhere else
+    can_overwrite = True
 
     def cache_need(self):
         s = self.spec
@@ -226,7 +241,7 @@ class PagedAttention(Mixer):
         return (splits(ctx.num_seqs, s.num_heads, s.num_kv_heads, ctx.max_ctx_len),)
 
     # ---- run
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, cache) -> None:
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, cache, overwrite: bool = False):
         s, rt = self.spec, self.runtime
         k = rt.kernels
         T = x.shape[0]
@@ -236,16 +251,16 @@ class PagedAttention(Mixer):
         if writes and not s.own_kv:
             raise ValueError("a layer without key and value projections must read another run step's cache")
         if self.prepared:
-            return self._prepared_attend(x, residual, ctx, cache)
+            return self._prepared_attend(x, residual, ctx, cache, overwrite)
         if self.bias_norm_gate:
-            return self._bias_norm_gate_attend(x, residual, ctx, cache)
+            return self._bias_norm_gate_attend(x, residual, ctx, cache, overwrite)
         if self.rotate_then_norm:
-            return self._rotate_norm_attend(x, residual, ctx, cache)
+            return self._rotate_norm_attend(x, residual, ctx, cache, overwrite)
         width = qw + self.kv_arrays * kw if writes else qw
         modified = s.softcap is not None or s.distance_bias is not None or s.chunk is not None or s.sink
         fused = self.position.fused_rotation()
         if fused is not None and fused[0] is not None and self._heads_from_the_product(x, ctx, cache, fused):
-            return self._attend(residual, ctx, cache)
+            return self._attend(residual, ctx, cache, overwrite=overwrite)
         split = getattr(k, "linear_partial", None)
         pending = None
         if split is not None and fused is not None and d % 4 == 0:
@@ -270,7 +285,7 @@ class PagedAttention(Mixer):
                             cache.page_size, s.scale, s.window, ctx.max_ctx_len, q_norm_w, k_norm_w, fused[0],
                             fused[1], norm.eps if norm is not None else 0.0,
                             norm.weight_offset if norm is not None else 0.0, writes, ctx.seq_rows):
-                return k.linear(att, self.o_proj, residual, residual=residual, defer=True)
+                return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
         if fused is None:
             # An encoding the kernels do not know: normalise head by head in
             # place, let the encoding transform q and k, then only copy and append.
@@ -291,9 +306,9 @@ class PagedAttention(Mixer):
             norm.weight_offset if norm is not None else 0.0,
             ctx.positions, ctx.seq_of_token, table if writes else None, nq, nkv, d, cache.page_size,
             ctx.seq_rows)
-        return self._attend(residual, ctx, cache)
+        return self._attend(residual, ctx, cache, overwrite=overwrite)
 
-    def _rotate_norm_attend(self, x, residual, ctx, cache):
+    def _rotate_norm_attend(self, x, residual, ctx, cache, overwrite=False):
         """The plain order: q | k | v product; per head rotation (with the encoding's
         amplitude), then the norm without a weight; append; attention; output product."""
         s, rt = self.spec, self.runtime
@@ -314,9 +329,9 @@ class PagedAttention(Mixer):
                               s.unit_norm_eps is not None, s.unit_norm_eps or 0.0, ctx.positions, ctx.seq_of_token,
                               ctx.tables[cache.group] if writes else None, nq, nkv, d, dv, cache.page_size,
                               ctx.seq_rows)
-        return self._attend(residual, ctx, cache)
+        return self._attend(residual, ctx, cache, overwrite=overwrite)
 
-    def _prepared_attend(self, x, residual, ctx, cache):
+    def _prepared_attend(self, x, residual, ctx, cache, overwrite=False):
         """q | k | v (| gates) from one product; biases, per-head norm, rotation and append in one
         kernel; attention with the maps of a head as heads of their own that share the head's
         values; the maps joined, normalised and gated; the output product."""
@@ -361,9 +376,9 @@ class PagedAttention(Mixer):
             k.differential_combine(att, gate, self.lam, s.differential_eps, 1.0 - float(s.differential), out,
                                    s.num_heads, dv, s.num_heads // s.num_kv_heads)
             att = out
-        return k.linear(att, self.o_proj, residual, residual=residual, defer=True)
+        return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
 
-    def _bias_norm_gate_attend(self, x, residual, ctx, cache):
+    def _bias_norm_gate_attend(self, x, residual, ctx, cache, overwrite=False):
         """q | k | v | gate from one product; biases, the norm over the whole q and k,
         a rotation if the encoding has one, and the append in one kernel; attention;
         the heads times sigmoid(gate); the output product."""
@@ -384,9 +399,9 @@ class PagedAttention(Mixer):
                                ctx.tables[cache.group] if writes else None, nq, nkv, d, dv, cache.page_size,
                                ctx.seq_rows)
         gate = proj[:, proj.shape[1] - self.gate_columns:] if self.gate_columns else None
-        return self._attend(residual, ctx, cache, gate)
+        return self._attend(residual, ctx, cache, gate, overwrite=overwrite)
 
-    def _attend(self, residual, ctx, cache, gate=None):
+    def _attend(self, residual, ctx, cache, gate=None, overwrite=False):
         """Attention over the cache from the step's q, then the output product, left
         for the next norm to add into the residual."""
         s, rt = self.spec, self.runtime
@@ -410,7 +425,7 @@ class PagedAttention(Mixer):
                     s.window, ctx.max_q_len, ctx.max_ctx_len, ctx.min_q_len, ctx.seq_rows, **extra)
         if gate is not None:
             k.sigmoid_gate(att, gate)
-        return k.linear(att, self.o_proj, residual, residual=residual, defer=True)
+        return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
 
     def _heads_from_the_product(self, x, ctx, cache, fused) -> bool:
         """Many rows on kernels that can do it: the q | k | v product normalises and

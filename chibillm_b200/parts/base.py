@@ -118,6 +118,12 @@ class PositionEncoding(Part):
     def fused_rotation(self):
         return None
 
+    def feature_order(self):
+        """The order in which a mixer has to put the features of its q and k heads when it binds its
+        weights (for every place the feature that stands there), so that ``fused_rotation`` rotates the
+        right pairs; None: the stored order."""
+        return None
+
     def step_table(self, ctx):
         """[tokens, rotary_dim] float32: the cosines, then the sines, of every token
         of the step, for kernels that rotate from a table; computed once per step
@@ -145,6 +151,10 @@ class Mixer(Part):
     # those products apply themselves.
     accepts_scaled_rows = False
 
+    # True: ``forward`` takes ``overwrite=True``, which says that ``residual`` holds nothing yet: the result
+    # is written over it instead of added to it (or is left pending).
+    can_overwrite = False
+
     def cache_need(self):
         return None
 
@@ -157,6 +167,10 @@ class FeedForward(Part):
     pending, as a mixer may)."""
 
     accepts_scaled_rows = False      # as for a mixer
+    can_overwrite = False            # as for a mixer
+    # a 32-bit vector that belongs to the result and that ``forward`` with ``overwrite=True`` leaves for the
+    # block to add (None: there is none)
+    output_bias = None
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
         raise NotImplementedError

@@ -7,7 +7,10 @@ needs), and no feed-forward at all.  With ``layer_scale`` each sublayer's result
 multiplied feature by feature by a learned vector before it joins the residual: the
 sublayer then adds into a 32-bit array of its own, and one kernel adds vector * array
 to the residual and writes the next norm's output (the block leaves that kernel
-pending, as it leaves a product pending otherwise).
+pending, as it leaves a product pending otherwise).  With norms on the sublayers' results
+(``mixer_out_norm``, ``feed_forward_out_norm``), a ``residual_scale`` or a weighted sum over all
+layers' results so far at the block's end (``depth_average``) the same kernel does those too, and adds
+up the partial sums of a sublayer's last product on the way (``SublayerEnd``).
 
 "parallel": one norm whose output both branches read,
 residual += scale * (mixer(norm(residual)) + feed_forward(norm(residual))), then an
@@ -51,6 +54,25 @@ class ScaledSum:
         return out
 
 
+class SublayerEnd:
+    """What a sublayer of a block with norms on its results leaves pending: with y the sublayer's sum (an
+    array, or the partial sums of its last product) + its bias,
+    residual += vec * y / rms(y) (or vec * y), then at a block's end the weighted sum over the results of
+    all blocks so far; the norm that follows can be done on the way."""
+
+    def __init__(self, kernels, delta, vec: torch.Tensor, eps, bias, depth=None):
+        self.kernels, self.delta, self.vec, self.eps, self.bias, self.depth = kernels, delta, vec, eps, bias, depth
+
+    def add_into(self, residual: torch.Tensor) -> None:
+        self.kernels.sublayer_end(residual, self.delta, self.vec, self.eps, self.bias, self.depth)
+
+    def finish_with_norm(self, residual: torch.Tensor, weight: torch.Tensor, eps: float, offset: float,
+                         out: torch.Tensor, scaled_ok: bool):
+        self.kernels.sublayer_end(residual, self.delta, self.vec, self.eps, self.bias, self.depth,
+                                  norm=(weight, eps, offset, out))
+        return out
+
+
 class PreNormBlock(Block):
     def __init__(self, layer, runtime: Runtime):
         self.layer = layer
@@ -71,6 +93,18 @@ class PreNormBlock(Block):
         if getattr(layer, "layer_scale", False):
             self.scale_names = (names["mixer_scale"],
                                 names["feed_forward_scale"] if self.feed_forward is not None else None)
+        # norms on the sublayers' results, a factor or a depth average: the order of SublayerEnd
+        self.out_norms = (layer.mixer_out_norm, layer.feed_forward_out_norm if self.feed_forward is not None else None)
+        self.out_norm_names = tuple(names[role] if n is not None else None for n, role in
+                                    zip(self.out_norms, ("mixer_out_norm", "feed_forward_out_norm")))
+        self.depth_name = names["depth_weights"] if layer.depth_average is not None else None
+        self.depth_weights: torch.Tensor = None
+        self.ends = any(n is not None for n in self.out_norms) or self.depth_name is not None \
+            or layer.residual_scale != 1.0
+        for n in self.out_norms:
+            if n is not None and (n.kind != "rmsnorm" or n.weight_offset != 0.0):
+                raise ValueError("a norm on a sublayer's result is an RMS norm with a plain weight")
+        self.end_vectors = [None, None]
 
     def expected_tensors(self) -> List[TensorSpec]:
         out: List[TensorSpec] = []
@@ -78,6 +112,10 @@ class PreNormBlock(Block):
             out.extend(p.expected_tensors())
         if self.scale_names is not None:
             out += [TensorSpec(n, (self.layer.mixer_norm.size,)) for n in self.scale_names if n is not None]
+        out += [TensorSpec(n, (self.layer.mixer_norm.size,)) for n in self.out_norm_names if n is not None]
+        if self.depth_name is not None:
+            earlier = self.layer.depth_average
+            out.append(TensorSpec(self.depth_name, (earlier + 1,), init=("normal", 1.0 / (earlier + 1), 0.1)))
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
@@ -87,6 +125,39 @@ class PreNormBlock(Block):
             self.mixer_scale = tensors[self.scale_names[0]].float().contiguous()
             if self.scale_names[1] is not None:
                 self.feed_forward_scale = tensors[self.scale_names[1]].float().contiguous()
+        if self.ends:
+            for i, (name, scale) in enumerate(zip(self.out_norm_names, (self.mixer_scale, self.feed_forward_scale))):
+                # residual_scale * scale * norm weight: one vector, made once in 32-bit
+                size, device = self.layer.mixer_norm.size, self.runtime.device
+                vec = torch.full((size,), float(self.layer.residual_scale), dtype=torch.float32, device=device)
+                for factor in (scale, tensors[name].float() if name is not None else None):
+                    vec = vec if factor is None else vec * factor
+                self.end_vectors[i] = vec.contiguous()
+        if self.depth_name is not None:
+            self.depth_weights = tensors[self.depth_name].float().contiguous()
+
+    def _ended(self, part, run, which: int, residual: torch.Tensor, ctx) -> SublayerEnd:
+        """Runs a sublayer into a 32-bit array of its own, or leaves its last product's partial sums."""
+        k = self.runtime.kernels
+        delta = ctx.workspace.get("block.delta." + ("mixer", "ff")[which], tuple(residual.shape), torch.float32)
+        if part.can_overwrite:
+            left = run(delta, {"overwrite": True})
+            bias = getattr(part, "output_bias", None)
+        else:
+            k.zero(delta)
+            left = run(delta, {})
+            bias = None
+        if left is not None:
+            if part.can_overwrite and hasattr(left, "partial"):
+                delta = left
+            else:
+                left.add_into(delta)
+        last = which == 1 or self.feed_forward is None
+        depth = None
+        if last and self.depth_name is not None:
+            depth = (ctx.shared["layer outputs"], self.layer.depth_average, self.depth_weights)
+        norm = self.out_norms[which]
+        return SublayerEnd(k, delta, self.end_vectors[which], None if norm is None else float(norm.eps), bias, depth)
 
     def _scaled(self, run, vec: torch.Tensor, residual: torch.Tensor, ctx, tag: str) -> ScaledSum:
         """Runs a sublayer into a 32-bit array of its own; what joins the residual is vec * that."""
@@ -118,7 +189,10 @@ class PreNormBlock(Block):
             mixed = ctx.workspace.get("block.conv", tuple(residual.shape), self.runtime.dtype)
             conv.forward(normed, mixed, ctx, conv_state)
             normed = mixed
-        if self.scale_names is not None:
+        if self.ends:
+            pending = self._ended(self.mixer, lambda acc, how: self.mixer.forward(normed, acc, ctx, cache, **how), 0,
+                                  residual, ctx)
+        elif self.scale_names is not None:
             pending = self._scaled(lambda acc: self.mixer.forward(normed, acc, ctx, cache), self.mixer_scale,
                                    residual, ctx, "mixer")
         else:
@@ -127,6 +201,9 @@ class PreNormBlock(Block):
             return pending
         normed = self.feed_forward_norm.forward_fused(residual, pending, x, self.feed_forward.accepts_scaled_rows)
         normed = x if normed is None else normed
+        if self.ends:
+            return self._ended(self.feed_forward, lambda acc, how: self.feed_forward.forward(normed, acc, ctx, **how), 1,
+                               residual, ctx)
         if self.scale_names is not None:
             return self._scaled(lambda acc: self.feed_forward.forward(normed, acc, ctx), self.feed_forward_scale,
                                 residual, ctx, "ff")

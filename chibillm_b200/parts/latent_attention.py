@@ -36,6 +36,8 @@ class LatentAttention(Mixer):
         self.names = names
         self.runtime = runtime
         self.position = make_position(spec.position, runtime)
+        if self.position.feature_order() is not None:
+            raise ValueError("latent attention rotates split halves")
         fused = self.position.fused_rotation()
         if fused is None or fused[0] is None or fused[1] != spec.rope_dim or getattr(self.position, "amplitude", 1.0) != 1.0:
             raise ValueError("latent attention needs a plain rotation over the whole rotated part")

@@ -20,7 +20,12 @@ scores from a softmax over all router outputs, chosen by score plus a correction
 within the best groups of outputs and weighted by the plain score times a constant;
 experts without tensors that return their input (their pairs are sorted into a bucket
 of their own whose rows are copies of the tokens' inputs, so the same combination
-weighs them); one more gated expert that every token uses."""
+weighs them); one more gated expert that every token uses, with an output gate per token if asked
+(its logit is one more row of the router's product); sigmoid scores; weights that multiply the experts'
+inputs (the first product's epilogue multiplies its 32-bit sums by the row's weight, which is the same).
+
+"mlp": a dense feed-forward without a gate; with "xielu" one kernel adds the bias and activates, and
+the second bias joins the sums of the second product."""
 from __future__ import annotations
 
 from typing import Dict, List
@@ -74,10 +79,14 @@ class GatedMLP(FeedForward):
 
     accepts_scaled_rows = True       # x goes to the gate | up product and nowhere else
 
+    @property
+    def can_overwrite(self):
+        return not self.spec.biases
+
     def launch_key(self, ctx):
         return ()
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, overwrite: bool = False):
         k = self.runtime.kernels
         T = x.shape[0]
         inter = self.spec.intermediate_size
@@ -91,11 +100,11 @@ class GatedMLP(FeedForward):
                 k.gated_activation(gate_up, self.bias_gate_up, act, self.spec.activation)
             if self.bias_down is not None:
                 k.add_row_vector(residual, self.bias_down)
-            return k.linear(act, self.down, residual, residual=residual, defer=True)
+            return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
         if self.gate_up_interleaved is not None:
             if not k.linear_swiglu(x, self.gate_up_interleaved, act):
                 raise RuntimeError("gated_mlp: the fused kernel refused a shape it was prepared for")
-            return k.linear(act, self.down, residual, residual=residual, defer=True)
+            return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
         split = getattr(k, "linear_partial", None)
         pending = split(x, self.gate_up) if split is not None else None
         if pending is not None:
@@ -104,7 +113,7 @@ class GatedMLP(FeedForward):
             gate_up = ctx.workspace.get("mlp.gate_up", (T, 2 * inter), self.runtime.dtype)
             k.linear(x, self.gate_up, gate_up)
             k.swiglu(gate_up, act)
-        return k.linear(act, self.down, residual, residual=residual, defer=True)
+        return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
 
 
 class DenseMLP(FeedForward):
@@ -112,40 +121,67 @@ class DenseMLP(FeedForward):
     activation is applied to the 32-bit sums of the first product (by the kernel
     that adds up a split product, or in place on the product's output)."""
 
-    ACTIVATIONS = ("gelu", "gelu_tanh", "silu", "relu")
+    ACTIVATIONS = ("gelu", "gelu_tanh", "silu", "relu", "xielu")
+    can_overwrite = True
 
     def __init__(self, spec, names: Dict[str, str], runtime: Runtime):
         if spec.activation not in self.ACTIVATIONS:
             raise ValueError(f"activation '{spec.activation}' is not supported by mlp; known: {self.ACTIVATIONS}")
+        if spec.biases and spec.activation != "xielu":
+            raise ValueError("mlp: biases belong to the activation 'xielu'")
         self.spec = spec
         self.names = names
         self.runtime = runtime
         self.up: torch.Tensor = None
         self.down: torch.Tensor = None
+        self.up_bias: torch.Tensor = None
+        self.output_bias: torch.Tensor = None
+        self.curvatures = (0.0, 0.0)     # xielu: softplus(p), 1/2 + softplus(q)
 
     def expected_tensors(self) -> List[TensorSpec]:
         s = self.spec
-        return [TensorSpec(self.names["up_proj"], (s.intermediate_size, s.hidden_size)),
-                TensorSpec(self.names["down_proj"], (s.hidden_size, s.intermediate_size))]
+        out = [TensorSpec(self.names["up_proj"], (s.intermediate_size, s.hidden_size)),
+               TensorSpec(self.names["down_proj"], (s.hidden_size, s.intermediate_size))]
+        if s.biases:
+            out += [TensorSpec(self.names["up_bias"], (s.intermediate_size,), init=("normal", 0.0, 0.1)),
+                    TensorSpec(self.names["down_bias"], (s.hidden_size,), init=("normal", 0.0, 0.1))]
+        if s.activation == "xielu":
+            out.append(TensorSpec(self.names["activation"], (2,), init=("uniform", -1.0, 1.0)))
+        return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.up = tensors[self.names["up_proj"]].contiguous()
         self.down = tensors[self.names["down_proj"]].contiguous()
+        if self.spec.biases:
+            self.up_bias = tensors[self.names["up_bias"]].float().contiguous()
+            self.output_bias = tensors[self.names["down_bias"]].float().contiguous()
+        if self.spec.activation == "xielu":
+            p, q = torch.nn.functional.softplus(tensors[self.names["activation"]].float()).tolist()
+            self.curvatures = (p, 0.5 + q)
 
     accepts_scaled_rows = True       # x goes to the up product and nowhere else
 
     def launch_key(self, ctx):
         return ()
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, overwrite: bool = False):
         k = self.runtime.kernels
         T = x.shape[0]
         act = ctx.workspace.get("mlp.act", (T, self.spec.intermediate_size), self.runtime.dtype)
-        fused = getattr(k, "linear_activation", None)
-        if fused is None or not fused(x, self.up, act, self.spec.activation):
-            k.linear(x, self.up, act)
-            k.activation(act, self.spec.activation)
-        return k.linear(act, self.down, residual, residual=residual, defer=True)
+        if self.spec.activation == "xielu":
+            up = k.linear_partial(x, self.up)          # partial sums, for the kernel that activates
+            if up is None:
+                up = act
+                k.linear(x, self.up, act)
+            k.bias_xielu(up, self.up_bias, act, *self.curvatures)
+            if not overwrite and self.output_bias is not None:
+                k.add_row_vector(residual, self.output_bias)
+        else:
+            fused = getattr(k, "linear_activation", None)
+            if fused is None or not fused(x, self.up, act, self.spec.activation):
+                k.linear(x, self.up, act)
+                k.activation(act, self.spec.activation)
+        return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
 
 
 class TableExperts(FeedForward):
@@ -278,12 +314,16 @@ class RoutedExperts(FeedForward):
         self.outputs = spec.num_experts + spec.identity_experts
         if not (0 < spec.top <= self.outputs):
             raise ValueError("routed_experts: 0 < top <= num_experts (+ identity_experts) is required")
-        if spec.scores not in ("softmax_top", "softmax_all"):
+        if spec.scores not in ("softmax_top", "softmax_all", "sigmoid"):
             raise ValueError(f"routed_experts: scores '{spec.scores}' is not supported")
+        if spec.weight_on_input and (not spec.gated or spec.identity_experts):
+            raise ValueError("routed_experts: weights on the inputs belong to gated experts, none of them an identity")
+        if spec.shared_output_gate and not spec.shared_size:
+            raise ValueError("routed_experts: an output gate needs a shared expert")
         if spec.scores == "softmax_top" and (spec.correction or spec.group_count != 1 or spec.identity_experts
                                              or spec.weight_scale != 1.0):
             raise ValueError("routed_experts: corrections, groups, identity experts and a weight scale belong "
-                             "to scores 'softmax_all'")
+                             "to scores 'softmax_all' and 'sigmoid'")
         if self.outputs % spec.group_count != 0 or not (0 < spec.group_keep <= spec.group_count) \
                 or spec.top > (self.outputs // spec.group_count) * spec.group_keep:
             raise ValueError("routed_experts: the router's outputs must form equal groups whose kept ones hold "
@@ -319,11 +359,17 @@ class RoutedExperts(FeedForward):
                     TensorSpec(self._name("expert_down", e), (s.hidden_size, s.intermediate_size))]
         if self.shared is not None:
             out += self.shared.expected_tensors()
+        if s.shared_output_gate:
+            out.append(TensorSpec(self.names["shared_output_gate"], (1, s.hidden_size), init=("normal", 0.0, 0.1)))
         return out
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         s = self.spec
         self.router = tensors[self.names["router"]].contiguous()
+        if s.shared_output_gate:
+            # the gate's logit is one more output of the router's product
+            gate = tensors[self.names["shared_output_gate"]].to(self.router.dtype)
+            self.router = torch.cat([self.router, gate], dim=0).contiguous()
         if s.correction:
             self.correction = tensors[self.names["correction"]].float().contiguous()
         if self.shared is not None:
@@ -351,32 +397,49 @@ class RoutedExperts(FeedForward):
     def launch_key(self, ctx):
         return ()
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx) -> None:
+    @property
+    def can_overwrite(self):
+        # the kernel that adds up the experts' outputs takes the shared expert's gated output along
+        return self.shared is None or self.spec.shared_output_gate
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, overwrite: bool = False):
         s, rt = self.spec, self.runtime
         k = rt.kernels
         T = x.shape[0]
         pairs = T * s.top
-        logits = ctx.workspace.get("router.logits", (T, self.outputs), torch.float32)
+        logits = ctx.workspace.get("router.logits", (T, self.router.shape[0]), torch.float32)
         k.linear(x, self.router, logits)
+        scores = logits[:, :self.outputs]
         chosen = ctx.workspace.get("router.chosen", (T, s.top), torch.int32)
         share = ctx.workspace.get("router.share", (T, s.top), torch.float32)
         buckets = self.up.shape[0]
         extra = {}
-        if s.scores == "softmax_all":
-            k.router_choose(logits, self.correction, chosen, share, s.group_count, s.group_keep, s.weight_scale,
-                            last_choice=buckets - 1)
+        if s.scores in ("softmax_all", "sigmoid"):
+            how = {"sigmoid": True} if s.scores == "sigmoid" else {}
+            k.router_choose(scores, self.correction, chosen, share, s.group_count, s.group_keep, s.weight_scale,
+                            last_choice=buckets - 1, **how)
             extra = {"gated": s.gated, "interleaved": self.interleaved, "identity": s.identity_experts}
         else:
-            k.router_top(logits, chosen, share)
+            k.router_top(scores, chosen, share)
             if s.gated:
                 extra = {"gated": True, "interleaved": self.interleaved}
+        if s.weight_on_input:
+            extra["weight_on_input"] = True
+        if overwrite:
+            extra["overwrite"] = True
+        if s.shared_output_gate:
+            # the shared expert first: its output, or its last product's partial sums, is gated and joined by
+            # the kernel that adds up the chosen experts' outputs
+            base = ctx.workspace.get("experts.shared", (T, s.hidden_size), torch.float32)
+            left = self.shared.forward(x, base, ctx, overwrite=True)
+            extra["base"] = (base if left is None else left, logits[:, self.outputs:])
         route = ctx.workspace.get("experts.route", (k.route_words(pairs, buckets),), torch.int32)
         act = ctx.workspace.get("experts.act", (pairs, s.intermediate_size), rt.dtype)
         y = ctx.workspace.get("experts.out", (pairs, s.hidden_size), torch.float32)
         sorted_x = ctx.workspace.get("experts.sorted", (pairs, s.hidden_size), rt.dtype)
         k.chosen_experts(x, chosen, share, self.up, self.down, residual, route, act, y, s.activation, sorted_x,
                          **extra)
-        if self.shared is not None:
+        if self.shared is not None and not s.shared_output_gate:
             return self.shared.forward(x, residual, ctx)
         return None
 

@@ -11,6 +11,9 @@ cosines and sines carry an amplitude other than one; the frequencies are then ma
 in 64-bit on the host and rounded once.  Kernels that rotate from ``inv_freq`` alone
 do not know the amplitude: a mixer asks ``amplitude`` and takes a kernel that does.
 
+``interleaved`` pairs (features 2i and 2i + 1) are the split-half rotation on reordered features: a mixer
+asks ``feature_order`` when it binds its weights and puts the rows of every q and k head in that order.
+
 "none": no position information inside the mixer.
 """
 from __future__ import annotations
@@ -92,6 +95,14 @@ class RotaryEncoding(PositionEncoding):
 
     def fused_rotation(self):
         return self.inv_freq, self.spec.rotary_dim
+
+    def feature_order(self):
+        """For every place of a head, the feature that is to stand there (None: as stored)."""
+        s = self.spec
+        if not s.interleaved:
+            return None
+        n = s.rotary_dim
+        return torch.tensor(list(range(0, n, 2)) + list(range(1, n, 2)) + list(range(n, s.head_dim)))
 
     def step_table(self, ctx):
         table_of = getattr(self.runtime.kernels, "rope_table", None)

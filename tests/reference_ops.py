@@ -331,10 +331,14 @@ class ReferenceKernels:
         share.copy_(torch.softmax(best, dim=-1))
 
     def chosen_experts(self, x, chosen, share, up, down, acc, route, act, y, kind, sorted_x=None, gated=False,
-                       interleaved=False, identity=0):
+                       interleaved=False, identity=0, weight_on_input=False, base=None, overwrite=False):
         self._count("chosen_experts")
         assert not interleaved
         F = down.shape[2]
+        if overwrite:
+            acc.zero_()
+        if base is not None:
+            acc.add_(torch.sigmoid(base[1].float()) * base[0])
         for t in range(x.shape[0]):
             total = torch.zeros_like(acc[t])
             for s in range(chosen.shape[1]):
@@ -343,8 +347,11 @@ class ReferenceKernels:
                     total += share[t, s] * x[t].float()
                     continue
                 z = up[e].float() @ x[t].float()
+                weight = share[t, s]
+                if weight_on_input:
+                    z, weight = z * weight, 1.0
                 hidden = (self._act(z[:F], kind) * z[F:]) if gated else self._act(z, kind)
-                total += share[t, s] * (down[e].float() @ hidden.to(x.dtype).float())
+                total += weight * (down[e].float() @ hidden.to(x.dtype).float())
             acc[t] += total
 
     # ---- the operations of hybrid_ops.cu
@@ -472,11 +479,12 @@ class ReferenceKernels:
         u = gate_up[:, n:].float().clamp(-limit, limit)
         out.copy_((g * torch.sigmoid(slope * g) * (u + 1.0)).to(out.dtype))
 
-    def router_choose(self, logits, correction, chosen, share, group_count, group_keep, scale, last_choice=None):
+    def router_choose(self, logits, correction, chosen, share, group_count, group_keep, scale, last_choice=None,
+                      sigmoid=False):
         self._count("router_choose")
         T, n = logits.shape
         top = chosen.shape[1]
-        s = torch.softmax(logits.float(), -1)
+        s = torch.sigmoid(logits.float()) if sigmoid else torch.softmax(logits.float(), -1)
         choice = s + correction if correction is not None else s.clone()
         if group_count > 1 and group_keep < group_count:
             per = n // group_count
@@ -496,6 +504,71 @@ class ReferenceKernels:
         if norm is not None:
             w, eps, offset, out = norm
             self.rmsnorm(residual, w, eps, offset, out)
+
+    # ---- the operations of linear_recurrence.cu and the sublayers' ends
+    def channel_delta(self, qkv, logits, beta, a_log, dt_bias, state, o, q_start, state_slots, heads, kv_heads, d, e,
+                      key_eps, q_scale, max_q_len):
+        self._count("channel_delta")
+        per = heads // kv_heads
+        kw = kv_heads * d
+        for s in range(state_slots.numel()):
+            slot = int(state_slots[s])
+            S = state[slot].clone()
+            for t in range(int(q_start[s]), int(q_start[s + 1])):
+                row = qkv[t].float()
+                q, k = row[:kw].view(kv_heads, d), row[kw:2 * kw].view(kv_heads, d)
+                v = row[2 * kw:].view(heads, e)
+                q = (q * torch.rsqrt((q * q).sum(-1, keepdim=True) + key_eps) * q_scale).repeat_interleave(per, 0)
+                k = (k * torch.rsqrt((k * k).sum(-1, keepdim=True) + key_eps)).repeat_interleave(per, 0)
+                step = torch.nn.functional.softplus(logits[t].float() + dt_bias).view(heads, d)
+                S = torch.exp(-torch.exp(a_log)[:, None] * step)[:, :, None] * S
+                u = torch.sigmoid(beta[t].float())[:, None] * (v - torch.einsum("hde,hd->he", S, k))
+                S = S + k[:, :, None] * u[:, None, :]
+                o[t] = torch.einsum("hde,hd->he", S, q).reshape(-1)
+            state[slot] = S
+
+    def decayed_attention(self, qkv, decay, state, o, q_start, state_slots, heads, d, e, max_q_len, activate=False):
+        self._count("decayed_attention")
+        kw = heads * d
+        for s in range(state_slots.numel()):
+            slot = int(state_slots[s])
+            S = state[slot].clone()
+            for t in range(int(q_start[s]), int(q_start[s + 1])):
+                row = qkv[t].float()
+                if activate:
+                    row = torch.nn.functional.silu(row)
+                q, k, v = row[:kw].view(heads, d), row[kw:2 * kw].view(heads, d), row[2 * kw:].view(heads, e)
+                S = decay[:, None, None] * S + k[:, :, None] * v[:, None, :]
+                o[t] = torch.einsum("hde,hd->he", S, q).reshape(-1)
+            state[slot] = S
+
+    def norm_then_gate(self, x, gate, weight, eps, out):
+        self._count("norm_then_gate")
+        y = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight
+        out.copy_((y * torch.sigmoid(gate.float())).to(out.dtype))
+
+    def bias_xielu(self, x, bias, out, curve_pos, curve_neg):
+        self._count("bias_xielu")
+        z = x.float() if bias is None else x.float() + bias
+        out.copy_(torch.where(z > 0, curve_pos * z * z, curve_neg * (torch.expm1(z) - z)).add(z / 2).to(out.dtype))
+
+    def sublayer_end(self, residual, delta, vec, eps, bias, depth=None, norm=None):
+        self._count("sublayer_end")
+        y = delta if bias is None else delta + bias
+        if eps is not None:
+            y = y * torch.rsqrt((y * y).mean(-1, keepdim=True) + eps)
+        residual.add_(vec * y)
+        if depth is not None:
+            outputs, earlier, weights = depth
+            if earlier < outputs.shape[0]:
+                outputs[earlier] = residual
+            total = weights[earlier] * residual
+            for j in range(earlier):
+                total = total + weights[j] * outputs[j]
+            residual.copy_(total)
+        if norm is not None:
+            w, n_eps, offset, out = norm
+            self.rmsnorm(residual, w, n_eps, offset, out)
 
     def side_gate(self, gate, tokens, table, offset, kind):
         e = table[tokens.long(), offset:offset + gate.shape[1]].float()
