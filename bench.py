@@ -15,8 +15,9 @@ its time, against the measured copy bandwidth; ``points`` decode at batch 1 and
 filled by real prefill steps for the end-to-end run and with random values for
 the device-timed runs (the work of a decode step does not depend on the values).
 
-``--design gitipel`` (or ``fokurax``, ``pitudra``, ``dogetar``) prints, instead of the record, prefill and decode
-of that design beside Qwen3 (Pitudra: beside Fokurax, Dogetar: beside Pitudra) at equal layer sizes, with the time of every kernel.
+``--design gitipel`` (or ``fokurax``, ``pitudra``, ``dogetar``, ``pafivik``) prints, instead of the record, prefill
+and decode of that design beside Qwen3 (Pitudra: beside Fokurax, Dogetar: beside Pitudra, Pafivik: beside Gitipel) at
+equal layer sizes, with the time of every kernel.
 
 ``--timeline`` prints, instead of the record, when the CTAs of every kernel of one
 decode step started, waited and ended.  ``--shape`` runs the same at the Qwen3-0.6B or
@@ -471,6 +472,33 @@ def dogetar_config(width, heads, kv_heads, dim, ff, vocab=32768):
             "loop": {"start": 1, "stop": 3, "times": 2}, "layers": [window, diff, par, diff]}
 
 
+def pafivik_config(width, heads, kv_heads, dim, ff, vocab=32768):
+    """Six layers, each with norms before and after its sublayers and a weighted sum over all results so far:
+    gated delta rule, gated delta rule, attention, linear attention with constant decays, gated delta rule,
+    attention.  The recurrences have heads of ``dim`` key and value channels over the whole width (the delta
+    rule: three taps, ranks of 64); attention has no window, every head is rotated.  Dense feed-forwards (xIELU
+    with biases) and routed ones (eight gated experts of half the dense size, two a token, and a gated shared
+    expert of the same size) in turn."""
+    dense = {"kind": "dense", "ff": ff}
+    experts = {"kind": "moe", "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2}, "router": {"experts": 8, "top": 2}}
+    n = width // dim
+
+    def delta(mlp):
+        return {"type": "channel_delta", "mlp": mlp,
+                "mixer": {"heads": n, "kv_heads": n, "dim": dim, "vdim": dim, "conv": 3, "decay_rank": 64, "gate_rank": 64}}
+
+    def attention(mlp):
+        return {"type": "attention", "mlp": mlp,
+                "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                          "rot": {"base": 1e6, "dims": dim}}}
+
+    lightning = {"type": "lightning", "mlp": experts,
+                 "mixer": {"heads": n, "dim": dim, "vdim": dim, "decay": [2.0 ** (-2.0 ** (-8.0 * h / n)) for h in range(n)]}}
+    return {"architecture": "Pafivik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
+            "residual_mult": 0.5,
+            "layers": [delta(dense), delta(experts), attention(dense), lightning, delta(dense), attention(experts)]}
+
+
 def qwen3_config_like(width, heads, kv_heads, dim, ff, layers=6, vocab=32768):
     cfg = dict(QWEN3_8B)
     cfg.update(num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv_heads,
@@ -541,11 +569,11 @@ def compare_designs(sizes, prompt_tokens, batch, held, steps, warmup, design="gi
     """Another design beside Qwen3 at equal layer sizes (six layer runs each, random weights);
     Pitudra beside Fokurax, the design nearest to it (routed experts, layers that read another
     layer's cache, a token input per layer); Dogetar beside Pitudra (a recurrent state, routed experts,
-    windows, sinks and gates)."""
+    windows, sinks and gates); Pafivik beside Gitipel (a delta rule beside attention)."""
     make = {"gitipel": gitipel_config, "fokurax": fokurax_config, "pitudra": pitudra_config,
-            "dogetar": dogetar_config}[design]
-    beside, make_other = {"pitudra": ("fokurax", fokurax_config),
-                          "dogetar": ("pitudra", pitudra_config)}.get(design, ("qwen3", qwen3_config_like))
+            "dogetar": dogetar_config, "pafivik": pafivik_config}[design]
+    beside, make_other = {"pitudra": ("fokurax", fokurax_config), "dogetar": ("pitudra", pitudra_config),
+                          "pafivik": ("gitipel", gitipel_config)}.get(design, ("qwen3", qwen3_config_like))
     result = {"metric": f"prefill and decode of {design.capitalize()} beside {beside.capitalize()} at equal layer sizes",
               "layer_runs": 6,
               "prompt_tokens": prompt_tokens, "decode_batch": batch, "decode_tokens_held": held, "dtype": "bf16",
@@ -638,9 +666,10 @@ def main() -> int:
     ap.add_argument("--check-tokens", type=int, default=0,
                     help="with --mixed-requests: also generate this many tokens of every request with the 32-bit "
                          "engine under two budgets and report how the runs agree")
-    ap.add_argument("--design", default=None, choices=["gitipel", "fokurax", "pitudra", "dogetar"],
+    ap.add_argument("--design", default=None, choices=["gitipel", "fokurax", "pitudra", "dogetar", "pafivik"],
                     help="instead of the record: prefill and decode of this design beside Qwen3 (pitudra: beside "
-                         "fokurax, dogetar: beside pitudra) at equal layer sizes (--design-sizes), with the time of every kernel")
+                         "fokurax, dogetar: beside pitudra, pafivik: beside gitipel) at equal layer sizes "
+                         "(--design-sizes), with the time of every kernel")
     ap.add_argument("--design-sizes", default="small,medium,large",
                     help="layer sizes for --design, with commas between them: " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--shape", default="qwen3-8b", choices=sorted(SHAPES),

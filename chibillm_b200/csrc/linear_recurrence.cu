@@ -8,14 +8,15 @@
 // Prompt portions go in chunks of 16 tokens (RC).  With G_t = g_1 .. g_t (row-wise products from the chunk's
 // start) and S_0 the state before the chunk, the u_t of a chunk solve a lower triangular system,
 //     u_t + b_t sum_{s<t} A_ts u_s = b_t (v_t - (G_t k_t)^T S_0),   A_ts = sum_c k_t[c] k_s[c] (g_{s+1} .. g_t)[c],
-// so that with M = (I + diag(b) A)^-1 diag(b)
-//     U = M (V - (G k) S_0),   o_t = (G_t q_t)^T S_0 + sum_{s<=t} B_ts u_s,   B_ts as A_ts with q_t for k_t,
+// so that with M = (I + diag(b) A)^-1 diag(b) and B_ts as A_ts with q_t for k_t (s <= t)
+//     U = M V - W S_0,               W = M (G k),
+//     O = (G q) S_0 + B U = B M V + Q S_0,   Q = (G q) - B W,
 //     S_end = diag(G_end) S_0 + sum_s (g_{s+1} .. g_end k_s) u_s^T.
 // All decays appear as products of factors from 0 to 1 (no quotients), so nothing overflows however strong
-// they are.  Without the delta rule U = V.  A first kernel makes, for every chunk and head at once, the rows
-// G k, G q, g_{s+1..end} k, the row G_end and the matrices M and B; a second kernel walks over a sequence's
-// chunks with a piece of S (all d rows of COLS columns) in registers.  A chunk that is not full has zero
-// rows for the tokens it lacks.
+// they are.  Without the delta rule U = V, Q = G q and O = B V + Q S_0.  A first kernel makes, for every chunk
+// and head at once, the rows W, Q, g_{s+1..end} k, the row G_end and the matrices M, B M; a second kernel walks
+// over a sequence's chunks with a piece of S (all d rows of some columns) in registers: two small products
+// with S_0 and V, then one into S.  A chunk that is not full has zero rows for the tokens it lacks.
 //
 // Few tokens a sequence (decode steps) run token by token in a kernel of their own.
 #define CHIBI_UNIT linear_recurrence
@@ -26,22 +27,28 @@ namespace chibi {
 
 constexpr int RC = 16;                                  // tokens of a chunk
 
-// Threads that share the inner products of the chunk kernel's first phase, and the pitch of a row of d
-// padded to DP: rows that a quarter of a warp reads together start on other banks.
-__host__ __device__ constexpr int rc_split(int DP, bool delta) { return delta ? DP / 32 : DP / 16; }
-__host__ __device__ constexpr int rc_pitch(int DP, bool delta)
-{
-    return DP + (rc_split(DP, delta) < 8 ? 4 * rc_split(DP, delta) : 4);
-}
-// A chunk's block in the scratch array, in floats: KE [RC][pitch] | QT [RC][pitch] | GE [DP] | B [RC][RC] and,
-// with the delta rule, | KT [RC][pitch] | M [RC][RC].
+// A chunk's block in the scratch array, in floats (d padded to DP): KE [RC][DP] | GE [DP] | Q [RC][DP] |
+// B M or B [RC][RC] and, with the delta rule, | -W [RC][DP] | M [RC][RC].
 __host__ __device__ constexpr int rc_block(int DP, bool delta)
 {
-    return (delta ? 3 : 2) * RC * rc_pitch(DP, delta) + DP + (delta ? 2 : 1) * RC * RC;
+    return (delta ? 3 : 2) * RC * DP + DP + (delta ? 2 : 1) * RC * RC;
 }
 
-__device__ __forceinline__ float lr_silu(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float lr_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+// silu, and the decay exp(rate * softplus(z)).  Beside bfloat16 activations CUDA's faster exponential and logarithm
+// (32-bit too, good to a few units of the last place of their results and to 2^-21 near one) are enough: an
+// input's own rounding is ten thousand times larger.
+template <typename TX> __device__ __forceinline__ float lr_silu(float z)
+{
+    if constexpr (sizeof(TX) == 2)
+        return __fdividef(z, 1.f + __expf(-z));
+    return z / (1.f + expf(-z));
+}
+template <typename TX> __device__ __forceinline__ float lr_decay(float rate, float z)
+{
+    if constexpr (sizeof(TX) == 2)
+        return __expf(rate * (z > 20.f ? z : __logf(1.f + __expf(z))));
+    return expf(rate * (z > 20.f ? z : log1pf(expf(z))));
+}
 
 struct RecurrenceParams {
     const void* q;             // [T, stride]: q of qk_heads * d columns
@@ -68,22 +75,32 @@ struct RecurrenceParams {
 };
 
 // ---------------------------------------------------------------- per chunk and head: what the chunk kernel needs
-// grid (chunks, heads, sequences), eight warps.  For a source token s a lane holds, for its channels, the
-// key times the decays since then, and walks over the later tokens t: its parts of A_ts and B_ts for all t
-// are folded over the lanes at once.
+// grid (chunks, heads, sequences), eight warps.  The inner products of a chunk's tokens come in tiles of four
+// sources s and four targets t, lanes along the channels.  Off the diagonal the sources are decayed to the
+// targets' first token and the targets from there, so that a tile is a plain product; on it the sources are
+// decayed token by token.  A tile's 32 sums over the lanes are folded together.
 template <int DP, bool DELTA, typename TX>
 __global__ void __launch_bounds__(256)
 recurrence_prepare_kernel(const RecurrenceParams p)
 {
+    // No trigger here: the chunk kernel's few blocks are to be dealt out to empty SMs, one to each.  Let in while
+    // this kernel's last blocks run, they crowd on the SMs that have room (2,048 tokens of 16 heads of 64: 0.18 ms
+    // became 0.47).
+#ifdef CHIBI_TIMELINE
     pdl_enter();
-    constexpr int P = rc_pitch(DP, DELTA), R = DP / 32;
+#else
+    pdl_wait();
+#endif
+    constexpr int R = DP / 32;
     extern __shared__ __align__(16) float sm[];
     float* ks = sm;                                     // [RC][DP]
     float* qs = ks + RC * DP;
     float* gs = qs + RC * DP;                           // [RC][DP] (delta rule)
-    __shared__ float As[RC][RC + 1];
-    __shared__ float Bs[RC][RC + 1];
-    __shared__ float bs[RC];
+    float* gg = gs + RC * DP;                           // [4][DP]: the decays' products over four tokens each
+    __shared__ __align__(16) float As[RC][RC];
+    __shared__ __align__(16) float Bs[RC][RC];
+    __shared__ __align__(16) float Ms[RC][RC];
+    __shared__ float bs[RC], power[RC + 1];
     const int h = blockIdx.y, seq = blockIdx.z;
     const int row0 = p.q_start[seq];
     const int base = blockIdx.x * RC;
@@ -94,38 +111,64 @@ recurrence_prepare_kernel(const RecurrenceParams p)
     const int d = p.d, kh = h / (p.heads / p.qk_heads);
     const TX* q = static_cast<const TX*>(p.q) + (size_t)(row0 + base) * p.stride + kh * d;
     const TX* k = static_cast<const TX*>(p.k) + (size_t)(row0 + base) * p.stride + kh * d;
-    float* out = p.scratch + ((size_t)((row0 / RC) + seq + blockIdx.x) * p.heads + h) * rc_block(DP, DELTA);
-    float* KE = out;
-    float* QT = KE + RC * P;
-    float* GE = QT + RC * P;
-    float* Bo = GE + DP;
-    float* KT = Bo + RC * RC;
-    float* Mo = KT + RC * P;
+    float* KE = p.scratch + ((size_t)((row0 / RC) + seq + blockIdx.x) * p.heads + h) * rc_block(DP, DELTA);
+    float* GE = KE + RC * DP;
+    float* Qo = GE + DP;
+    float* No = Qo + RC * DP;                           // B M, or B
+    float* Wo = No + RC * RC;
+    float* Mo = Wo + RC * DP;
     const float rate = DELTA ? -expf(p.a_log[h]) : 0.f;
-    const float decay = DELTA ? 1.f : p.decay[h];
 
-    for (int i = tid; i < RC * DP; i += 256) {
-        const int t = i / DP, c = i - t * DP;
-        float kv = 0.f, qv = 0.f, g = 1.f;
-        if (t < n && c < d) {
-            kv = to_f32(k[(size_t)t * p.stride + c]);
-            qv = to_f32(q[(size_t)t * p.stride + c]);
-            if (p.activate)
-                kv = lr_silu(kv), qv = lr_silu(qv);
-            if (DELTA)
-                g = expf(rate * lr_softplus(p.logits[(size_t)(row0 + base + t) * p.logit_stride + h * d + c]
-                                            + p.dt_bias[h * d + c]));
+    // ---- the chunk's keys, queries and decays
+    {
+        constexpr int PER = RC * DP / 256;              // a thread's values: the channel is the same for all (or two)
+        TX kr[PER], qr[PER];
+        float zr[PER];
+#pragma unroll
+        for (int u = 0; u < PER; ++u) {
+            const int i = tid + 256 * u, t = i / DP, c = i - t * DP;
+            kr[u] = qr[u] = from_f32<TX>(0.f);
+            zr[u] = 0.f;
+            if (t < n && c < d) {
+                kr[u] = k[(size_t)t * p.stride + c];
+                qr[u] = q[(size_t)t * p.stride + c];
+                if (DELTA)
+                    zr[u] = p.logits[(size_t)(row0 + base + t) * p.logit_stride + h * d + c] + p.dt_bias[h * d + c];
+            }
         }
-        ks[i] = kv;
-        qs[i] = qv;
-        if (DELTA)
-            gs[i] = g;
+#pragma unroll
+        for (int u = 0; u < PER; ++u) {
+            const int i = tid + 256 * u, t = i / DP, c = i - t * DP;
+            float kv = to_f32(kr[u]), qv = to_f32(qr[u]);
+            if (p.activate)
+                kv = lr_silu<TX>(kv), qv = lr_silu<TX>(qv);     // (silu(0) is 0)
+            ks[i] = kv;
+            qs[i] = qv;
+            if (DELTA)
+                gs[i] = t < n && c < d ? lr_decay<TX>(rate, zr[u]) : 1.f;
+        }
     }
-    if (DELTA && tid < RC)
-        bs[tid] = tid < n ? 1.f / (1.f + expf(-to_f32(static_cast<const TX*>(p.beta)[(size_t)(row0 + base + tid)
-                                                                                    * p.beta_stride + h]))) : 0.f;
+    if (tid < RC) {
+        if (DELTA) {
+            bs[tid] = tid < n ? 1.f / (1.f + expf(-to_f32(static_cast<const TX*>(p.beta)[(size_t)(row0 + base + tid)
+                                                                                        * p.beta_stride + h]))) : 0.f;
+        } else {
+            float v = 1.f;
+            for (int i = 0; i < tid; ++i)
+                v *= p.decay[h];
+            power[tid] = v;
+            if (tid == RC - 1)
+                power[RC] = v * p.decay[h];
+        }
+    }
+    if (tid < RC * RC / 4) {                            // (what lies above the diagonal)
+        reinterpret_cast<float4*>(&As[0][0])[tid] = make_float4(0.f, 0.f, 0.f, 0.f);
+        reinterpret_cast<float4*>(&Bs[0][0])[tid] = make_float4(0.f, 0.f, 0.f, 0.f);
+        reinterpret_cast<float4*>(&Ms[0][0])[tid] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     __syncthreads();
-    if (DELTA) {                                        // unit keys and queries: two tokens to a warp
+    if (DELTA) {
+        // unit keys and queries: two tokens to a warp
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
             const int t = warp + 8 * u;
@@ -144,51 +187,77 @@ recurrence_prepare_kernel(const RecurrenceParams p)
                 qs[t * DP + lane + 32 * i] *= iq;
             }
         }
+        for (int i = tid; i < 4 * DP; i += 256) {
+            const int b = i / DP, c = i - b * DP;
+            const float* g = gs + 4 * b * DP + c;
+            gg[i] = g[0] * g[DP] * (g[2 * DP] * g[3 * DP]);
+        }
         __syncthreads();
     }
-    // decays from the chunk's start, a thread to a channel
-    for (int c = tid; c < DP; c += 256) {
-        float g = 1.f;
-#pragma unroll
-        for (int t = 0; t < RC; ++t) {
-            g *= DELTA ? gs[t * DP + c] : (t < n ? decay : 1.f);
-            QT[t * P + c] = qs[t * DP + c] * g;
-            if (DELTA)
-                KT[t * P + c] = ks[t * DP + c] * g;
-        }
-        GE[c] = g;
-    }
-    // a warp takes the source tokens `warp` and 15 - `warp`
+    // ---- tiles of inner products: (block of targets, block of sources); warps 6 and 7 take two on the diagonal
 #pragma unroll 1
-    for (int u = 0; u < 2; ++u) {
-        const int s = u ? RC - 1 - warp : warp;
-        float w[R], acc[2 * RC];                        // [t]: B_ts, A_ts
+    for (int item = warp; item < 10; item = item < 6 ? 10 : item + 2) {
+        const int I = item < 6 ? (item == 0 ? 1 : item < 3 ? 2 : 3) : item - 6;
+        const int J = item < 6 ? (item == 0 ? 0 : item < 3 ? item - 1 : item - 3) : item - 6;
+        float acc[32];                                  // [4 t + s]: A, then B
 #pragma unroll
-        for (int i = 0; i < R; ++i)
-            w[i] = ks[s * DP + lane + 32 * i];
+        for (int i = 0; i < 32; ++i)
+            acc[i] = 0.f;
 #pragma unroll
-        for (int t = 0; t < RC; ++t) {
-            float b = 0.f, a = 0.f;
-            if (t >= s) {
+        for (int r = 0; r < R; ++r) {
+            const int c = lane + 32 * r;
+            float w[4];
 #pragma unroll
-                for (int i = 0; i < R; ++i) {
-                    const int c = t * DP + lane + 32 * i;
-                    if (t > s)
-                        w[i] *= DELTA ? gs[c] : (t < n ? decay : 1.f);
-                    b = fmaf(qs[c], w[i], b);
-                    if (DELTA)
-                        a = fmaf(ks[c], w[i], a);
+            for (int s = 0; s < 4; ++s)
+                w[s] = ks[(4 * J + s) * DP + c];
+            if (!DELTA) {
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    const float qv = qs[(4 * I + t) * DP + c];
+#pragma unroll
+                    for (int s = 0; s < 4; ++s)
+                        acc[16 + 4 * t + s] = fmaf(qv, w[s], acc[16 + 4 * t + s]);
+                }
+            } else if (item < 6) {
+                float f = 1.f;                          // from the end of the sources' block to the targets' first token
+                for (int b = J + 1; b < I; ++b)
+                    f *= gg[b * DP + c];
+#pragma unroll
+                for (int s = 3; s >= 0; --s) {
+                    w[s] *= f;
+                    if (s > 0)
+                        f *= gs[(4 * J + s) * DP + c];
+                }
+                f = 1.f;
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    const int at = (4 * I + t) * DP + c;
+                    f *= gs[at];
+                    const float kv = ks[at] * f, qv = qs[at] * f;
+#pragma unroll
+                    for (int s = 0; s < 4; ++s) {
+                        acc[4 * t + s] = fmaf(kv, w[s], acc[4 * t + s]);
+                        acc[16 + 4 * t + s] = fmaf(qv, w[s], acc[16 + 4 * t + s]);
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int t = 0; t < 4; ++t) {
+                    const int at = (4 * I + t) * DP + c;
+                    const float kv = ks[at], qv = qs[at], g = gs[at];
+#pragma unroll
+                    for (int s = 0; s < t; ++s) {
+                        w[s] *= g;
+                        acc[4 * t + s] = fmaf(kv, w[s], acc[4 * t + s]);
+                        acc[16 + 4 * t + s] = fmaf(qv, w[s], acc[16 + 4 * t + s]);
+                    }
+                    acc[16 + 4 * t + t] = fmaf(qv, w[t], acc[16 + 4 * t + t]);
                 }
             }
-            acc[t] = b;
-            acc[RC + t] = a;
         }
-#pragma unroll
-        for (int i = 0; i < R; ++i)
-            KE[s * P + lane + 32 * i] = w[i];
         // fold: after the steps 16, 8, 4, 2, 1 lane l holds the sum over all lanes of value l
 #pragma unroll
-        for (int half = RC, o = 16; half >= 1; half >>= 1, o >>= 1) {
+        for (int half = 16, o = 16; half >= 1; half >>= 1, o >>= 1) {
             const bool upper = (lane & o) != 0;
 #pragma unroll
             for (int i = 0; i < half; ++i) {
@@ -197,24 +266,103 @@ recurrence_prepare_kernel(const RecurrenceParams p)
                 acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
             }
         }
-        if (lane < RC)
-            Bs[lane][s] = acc[0];
-        else
-            As[lane - RC][s] = acc[0];
+        const int t = 4 * I + ((lane >> 2) & 3), s = 4 * J + (lane & 3);
+        if (lane < 16) {
+            if (DELTA)
+                As[t][s] = acc[0];
+        } else if (t >= s) {
+            Bs[t][s] = DELTA ? acc[0] : acc[0] * power[t - s];
+        }
     }
     __syncthreads();
-    Bo[tid] = Bs[tid / RC][tid % RC];                   // (256 threads, 16 x 16 values)
-    if (DELTA && tid < RC) {
-        // column tid of M: forward substitution
+    if (!DELTA) {
+        No[tid] = Bs[tid / RC][tid % RC];               // (256 threads, 16 x 16 values)
+        for (int c = tid; c < DP; c += 256) {
+#pragma unroll
+            for (int t = 0; t < RC; ++t) {
+                Qo[t * DP + c] = qs[t * DP + c] * power[t + 1];
+                KE[t * DP + c] = t < n ? ks[t * DP + c] * power[n - 1 - t] : 0.f;
+            }
+            GE[c] = power[n];
+        }
+        return;
+    }
+    // ---- M: a column to a thread, forward substitution; meanwhile the other warps decay the keys to the chunk's end
+    if (tid < RC) {
         float m[RC];
 #pragma unroll
         for (int t = 0; t < RC; ++t) {
-            float v = t == tid ? 1.f : 0.f;
+            float v0 = t == tid ? 1.f : 0.f, v1 = 0.f;
 #pragma unroll
-            for (int s = 0; s < t; ++s)
-                v = fmaf(-As[t][s], m[s], v);
-            m[t] = bs[t] * v;
-            Mo[t * RC + tid] = m[t];
+            for (int s = 0; s < t; ++s) {
+                if (s & 1)
+                    v1 = fmaf(-As[t][s], m[s], v1);
+                else
+                    v0 = fmaf(-As[t][s], m[s], v0);
+            }
+            m[t] = bs[t] * (v0 + v1);
+            Ms[t][tid] = m[t];
+        }
+    } else if (tid >= 32) {
+        for (int c = tid - 32; c < DP; c += 224) {
+            float f = 1.f;
+#pragma unroll
+            for (int t = RC - 1; t >= 0; --t) {
+                KE[t * DP + c] = ks[t * DP + c] * f;
+                f *= gs[t * DP + c];
+            }
+            GE[c] = f;
+        }
+    }
+    __syncthreads();
+    {
+        const int t = tid / RC, j = tid % RC;
+        float v = 0.f;
+#pragma unroll
+        for (int s = 0; s < RC; ++s)
+            v = fmaf(Bs[t][s], Ms[s][j], v);
+        No[tid] = v;
+        Mo[tid] = Ms[t][j];
+    }
+    // ---- W and Q, a channel to a thread
+    for (int c = tid; c < DP; c += 256) {
+        float w[RC], g[RC];
+        float f = 1.f;
+#pragma unroll
+        for (int t = 0; t < RC; ++t) {
+            f *= gs[t * DP + c];
+            g[t] = f;
+        }
+        {
+            float kt[RC];
+#pragma unroll
+            for (int t = 0; t < RC; ++t) {
+                kt[t] = ks[t * DP + c] * g[t];
+                float v = 0.f;
+#pragma unroll
+                for (int s4 = 0; s4 <= t; s4 += 4) {
+                    const float4 m = *reinterpret_cast<const float4*>(&Ms[t][s4]);
+                    v = fmaf(m.x, kt[s4], v);
+                    if (s4 + 1 <= t) v = fmaf(m.y, kt[s4 + 1], v);
+                    if (s4 + 2 <= t) v = fmaf(m.z, kt[s4 + 2], v);
+                    if (s4 + 3 <= t) v = fmaf(m.w, kt[s4 + 3], v);
+                }
+                w[t] = v;
+                Wo[t * DP + c] = -v;
+            }
+        }
+#pragma unroll
+        for (int t = 0; t < RC; ++t) {
+            float v = qs[t * DP + c] * g[t];
+#pragma unroll
+            for (int s4 = 0; s4 <= t; s4 += 4) {
+                const float4 m = *reinterpret_cast<const float4*>(&Bs[t][s4]);
+                v = fmaf(-m.x, w[s4], v);
+                if (s4 + 1 <= t) v = fmaf(-m.y, w[s4 + 1], v);
+                if (s4 + 2 <= t) v = fmaf(-m.z, w[s4 + 2], v);
+                if (s4 + 3 <= t) v = fmaf(-m.w, w[s4 + 3], v);
+            }
+            Qo[t * DP + c] = v;
         }
     }
 }
@@ -226,65 +374,86 @@ __device__ __forceinline__ void rc_copy16(float* dst, const float* src)
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(a), "l"(src) : "memory");
 }
 
-// grid (blocks of COLS value columns, heads, sequences), DP * COLS / 16 threads.  A thread owns 4 x 4 elements
-// of S (rows r0 .., columns c0 ..) in registers; a copy lies in shared memory, column by column, for the
-// first phase, in which KS neighbouring threads share a tile of 4 tokens x 4 columns of (G k) S_0 or (G q) S_0
-// (each its part of the d rows) and fold their sums.
-template <int DP, int COLS, bool DELTA, typename TX>
-__global__ void __launch_bounds__(DP * COLS / 16)
+// Two 32-bit values in one 64-bit register, and the multiply-add that takes two such pairs (each half rounded
+// like fmaf).
+__device__ __forceinline__ uint64_t rc_pair(float a, float b)
+{
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ float2 rc_halves(uint64_t v)
+{
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ uint64_t rc_fma2(uint64_t a, uint64_t b, uint64_t c)
+{
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t rc_mul2(uint64_t a, uint64_t b)
+{
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
+// grid (blocks of COLS value columns, heads, sequences).  A thread owns RT rows (runs of four) of CT columns of S
+// in registers, two neighbouring rows to a pair, DP / RT threads of a warp lie side by side along the rows, and the
+// chunk's rows come from shared memory.  The sums over the rows are spread over those threads and folded at the end of a product, all of its
+// values together.  Small pieces of S and many threads: a sequence's chunks come one after the other, so the
+// time of a chunk counts, and with a few columns a block every SM has one.
+template <int DP, int RT, int CT, int COLS, bool DELTA, typename TX>
+__global__ void __launch_bounds__((DP / RT) * (COLS / CT))
 chunk_recurrence_kernel(const RecurrenceParams p)
 {
-    constexpr int NT = DP * COLS / 16, P = rc_pitch(DP, DELTA), KS = rc_split(DP, DELTA), BLOCK = rc_block(DP, DELTA);
-    constexpr int CP = COLS + 4;                        // pitch of the chunk's small arrays
-    constexpr int CG = COLS / 4;                        // groups of four columns
-    constexpr int OWN = 16 / KS;                        // sums a thread is left with after the fold
-    static_assert(NT % 32 == 0 && KS >= 1 && KS <= 16 && DP % (4 * KS) == 0, "sizes");
+    constexpr int L = DP / RT;                          // threads along the rows
+    constexpr int NT = L * (COLS / CT), BLOCK = rc_block(DP, DELTA), CP = COLS + 4;
+    constexpr int VR = L >= RC ? 1 : RC / L;            // rows of V (tokens) that a thread owns for the products
+    constexpr int SUMS = RC * CT, OWN = SUMS / L;       // a product's values, and those that a thread is left with
+    constexpr int RUNS = RT / 4, RUN_STEP = DP / RUNS;  // its rows: runs r0 + RUN_STEP i .. + 3
+    static_assert(L <= 32 && 32 % L == 0 && NT % 32 == 0 && RT % 4 == 0 && OWN >= 1, "sizes");
 #ifdef CHIBI_TIMELINE
     pdl_enter();
 #endif
     extern __shared__ __align__(16) float sm[];
     float* bufs = sm;                                   // two chunks
-    float* Sc = bufs + 2 * BLOCK;                       // [COLS][P]
-    float* Us = Sc + COLS * P;                          // [RC][CP]
-    float* Os = Us + RC * CP;                           // [RC][CP]
-    float* Rs = Os + RC * CP;                           // [RC][CP] (delta rule)
+    float* Us = bufs + 2 * BLOCK;                       // [RC][CP]
     const int h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
     const int d = p.d, e = p.e;
-    const int col0 = blockIdx.x * COLS;
     const int row0 = p.q_start[seq];
     const int len = p.q_start[seq + 1] - row0;
     if (len <= 0)
         return;
-    const int r0 = 4 * (tid % (DP / 4)), c0 = 4 * (tid / (DP / 4));
+    const int lr = tid % L, c0 = CT * (tid / L), r0 = 4 * lr;
+    const int col = blockIdx.x * COLS + c0;             // the thread's first column
     float* st = p.state + ((size_t)p.slots[seq] * p.heads + h) * d * e;
-    float S[4][4];                                      // [column][row]
+    uint64_t S[RT / 2][CT];
     // (the state is what an earlier step left: fetched before the kernel ahead is through)
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < RT / 2; ++i) {
+        const int r = r0 + RUN_STEP * (i / 2) + 2 * (i % 2);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            S[j][i] = (r0 + i < d && col0 + c0 + j < e) ? st[(size_t)(r0 + i) * e + col0 + c0 + j] : 0.f;
+        for (int j = 0; j < CT; ++j)
+            S[i][j] = rc_pair((r < d && col + j < e) ? st[(size_t)r * e + col + j] : 0.f,
+                              (r + 1 < d && col + j < e) ? st[(size_t)(r + 1) * e + col + j] : 0.f);
+    }
 #ifndef CHIBI_TIMELINE
     pdl_wait();
 #endif
-    // the tile of the first phase, and the sums of it that this thread is left with
-    const int ks = tid % KS, tile = tid / KS;
-    const int tg = tile & 3, cg = (tile >> 2) % CG;
-    const bool keys = DELTA && tile >= 4 * CG;          // this thread works on (G k) S_0, else on (G q) S_0
-    const int first = ks * OWN;                         // values first .. first + OWN - 1 of the tile's 16 (token-major)
-    const TX* v = static_cast<const TX*>(p.v) + (size_t)row0 * p.stride + (size_t)h * e + col0;
-    const bool takes_v = !DELTA || keys;
-    float vn[OWN];
+    const TX* v = static_cast<const TX*>(p.v) + (size_t)row0 * p.stride + (size_t)h * e + col;
+    TX vn[VR][CT];                                      // on their way: nothing is done with them before their chunk
     auto fetch_v = [&](int base) {
 #pragma unroll
-        for (int m = 0; m < OWN; ++m) {
-            const int t = tg + 4 * ((first + m) >> 2), c = cg + CG * ((first + m) & 3);
-            vn[m] = 0.f;
-            if (takes_v && base + t < len && col0 + c < e) {
-                vn[m] = to_f32(v[(size_t)(base + t) * p.stride + c]);
-                if (p.activate)
-                    vn[m] = lr_silu(vn[m]);
-            }
+        for (int i = 0; i < VR; ++i) {
+            const int t = lr + L * i;
+#pragma unroll
+            for (int j = 0; j < CT; ++j)
+                vn[i][j] = (t < RC && base + t < len && col + j < e) ? v[(size_t)(base + t) * p.stride + j]
+                                                                    : from_f32<TX>(0.f);
         }
     };
     const float* chunk_src = p.scratch + ((size_t)(row0 / RC + seq) * p.heads + h) * BLOCK;
@@ -296,9 +465,6 @@ chunk_recurrence_kernel(const RecurrenceParams p)
     };
     fetch(0, bufs);
     fetch_v(0);
-#pragma unroll
-    for (int j = 0; j < 4; ++j)
-        *reinterpret_cast<float4*>(Sc + (c0 + j) * P + r0) = make_float4(S[j][0], S[j][1], S[j][2], S[j][3]);
 
     const int chunks = (len + RC - 1) / RC;
     for (int c = 0; c < chunks; ++c) {
@@ -307,48 +473,57 @@ chunk_recurrence_kernel(const RecurrenceParams p)
         if (c + 1 < chunks)
             fetch(c + 1, bufs + ((c + 1) & 1) * BLOCK);
         const float* KE = bufs + (c & 1) * BLOCK;
-        const float* QT = KE + RC * P;
-        const float* GE = QT + RC * P;
-        const float* B = GE + DP;
-        const float* KT = B + RC * RC;
-        const float* M = KT + RC * P;
+        const float* GE = KE + RC * DP;
+        const float* Q = GE + DP;
+        const float* NO = Q + RC * DP;
+        const float* W = NO + RC * RC;
+        const float* M = W + RC * DP;
         const int base = c * RC;
-        float v_now[OWN];
+        float vt[VR][CT];
 #pragma unroll
-        for (int m = 0; m < OWN; ++m)
-            v_now[m] = vn[m];
+        for (int i = 0; i < VR; ++i)
+#pragma unroll
+            for (int j = 0; j < CT; ++j) {
+                vt[i][j] = to_f32(vn[i][j]);
+                if (p.activate)
+                    vt[i][j] = lr_silu<TX>(vt[i][j]);
+            }
         if (c + 1 < chunks)
             fetch_v(base + RC);
-        // ---- (G q) S_0 and (G k) S_0
-        {
-            float acc[16];
+        // A S_0 + N V, folded: thread lr ends with values lr OWN .. of the [token][column] tile
+        auto product = [&](const float* A, const float* N, float (&acc)[SUMS]) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i)
-                acc[i] = 0.f;
-            const float* a_rows = (keys ? KT : QT) + tg * P + 4 * ks;
-            const float* b_rows = Sc + cg * P + 4 * ks;
-#pragma unroll 4
-            for (int k4 = 0; k4 < DP / (4 * KS); ++k4) {
-                float4 a[4], b[4];
+            for (int t = 0; t < RC; ++t) {
+                uint64_t pair[CT];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    a[i] = *reinterpret_cast<const float4*>(a_rows + 4 * i * P + 4 * KS * k4);
-                    b[i] = *reinterpret_cast<const float4*>(b_rows + CG * i * P + 4 * KS * k4);
+                for (int u = 0; u < RUNS; ++u) {
+                    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(A + t * DP + r0 + RUN_STEP * u);
+#pragma unroll
+                    for (int j = 0; j < CT; ++j) {
+                        pair[j] = u == 0 ? rc_mul2(a.x, S[0][j]) : rc_fma2(a.x, S[2 * u][j], pair[j]);
+                        pair[j] = rc_fma2(a.y, S[2 * u + 1][j], pair[j]);
+                    }
+                }
+                float s[CT];
+#pragma unroll
+                for (int j = 0; j < CT; ++j) {
+                    const float2 halves = rc_halves(pair[j]);
+                    s[j] = halves.x + halves.y;
                 }
 #pragma unroll
-                for (int i = 0; i < 4; ++i)
+                for (int i = 0; i < VR; ++i) {
+                    const float m = L <= RC || lr < RC ? N[t * RC + lr + L * i] : 0.f;
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        float s = acc[4 * i + j];
-                        s = fmaf(a[i].x, b[j].x, s);
-                        s = fmaf(a[i].y, b[j].y, s);
-                        s = fmaf(a[i].z, b[j].z, s);
-                        acc[4 * i + j] = fmaf(a[i].w, b[j].w, s);
-                    }
+                    for (int j = 0; j < CT; ++j)
+                        s[j] = fmaf(m, vt[i][j], s[j]);
+                }
+#pragma unroll
+                for (int j = 0; j < CT; ++j)
+                    acc[CT * t + j] = s[j];
             }
 #pragma unroll
-            for (int o = KS / 2, half = 8; o >= 1; o >>= 1, half >>= 1) {
-                const bool upper = (ks & o) != 0;
+            for (int o = L / 2, half = SUMS / 2; o >= 1; o >>= 1, half >>= 1) {
+                const bool upper = (lr & o) != 0;
 #pragma unroll
                 for (int i = 0; i < half; ++i) {
                     const float send = upper ? acc[i] : acc[i + half];
@@ -356,84 +531,78 @@ chunk_recurrence_kernel(const RecurrenceParams p)
                     acc[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
                 }
             }
+        };
+        if (DELTA) {
+            float acc[SUMS];
+            product(W, M, acc);
 #pragma unroll
-            for (int m = 0; m < OWN; ++m) {
-                const int t = tg + 4 * ((first + m) >> 2), cc = cg + CG * ((first + m) & 3);
-                if (keys) {
-                    Rs[t * CP + cc] = v_now[m] - acc[m];
-                } else {
-                    Os[t * CP + cc] = acc[m];
-                    if (!DELTA)
-                        Us[t * CP + cc] = v_now[m];
-                }
-            }
+            for (int i = 0; i < OWN; ++i)
+                Us[((lr * OWN + i) / CT) * CP + c0 + (lr * OWN + i) % CT] = acc[i];
+        } else {
+#pragma unroll
+            for (int i = 0; i < VR; ++i)
+#pragma unroll
+                for (int j = 0; j < CT; ++j)
+                    if (lr + L * i < RC)
+                        Us[(lr + L * i) * CP + c0 + j] = vt[i][j];
         }
         __syncthreads();
-        // ---- U = M R, four columns of a token to a thread
-        if (DELTA) {
-            for (int i = tid; i < RC * CG; i += NT) {
-                const int t = i / CG, cc = 4 * (i - t * CG);
-                float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-                for (int s = 0; s < RC; ++s) {
-                    const float m = M[t * RC + s];
-                    const float4 r = *reinterpret_cast<const float4*>(Rs + s * CP + cc);
-                    u.x = fmaf(m, r.x, u.x), u.y = fmaf(m, r.y, u.y), u.z = fmaf(m, r.z, u.z), u.w = fmaf(m, r.w, u.w);
-                }
-                *reinterpret_cast<float4*>(Us + t * CP + cc) = u;
-            }
-            __syncthreads();
-        }
-        // ---- o = (G q) S_0 + B U
-        for (int i = NT - 1 - tid; i < RC * CG; i += NT) {
-            const int t = i / CG, cc = 4 * (i - t * CG);
-            if (base + t >= len)
-                continue;
-            float4 u = *reinterpret_cast<const float4*>(Os + t * CP + cc);
-#pragma unroll
-            for (int s = 0; s < RC; ++s) {
-                const float m = B[t * RC + s];
-                const float4 r = *reinterpret_cast<const float4*>(Us + s * CP + cc);
-                u.x = fmaf(m, r.x, u.x), u.y = fmaf(m, r.y, u.y), u.z = fmaf(m, r.z, u.z), u.w = fmaf(m, r.w, u.w);
-            }
-            float* dst = p.o + (size_t)(row0 + base + t) * p.heads * e + (size_t)h * e + col0 + cc;
-            const float out[4] = { u.x, u.y, u.z, u.w };
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                if (col0 + cc + j < e)
-                    dst[j] = out[j];
-        }
-        // ---- S = diag(G_end) S_0 + KE^T U
         {
-            const float4 g = *reinterpret_cast<const float4*>(GE + r0);
+            float acc[SUMS];
+            product(Q, NO, acc);
 #pragma unroll
-            for (int j = 0; j < 4; ++j)
-                S[j][0] *= g.x, S[j][1] *= g.y, S[j][2] *= g.z, S[j][3] *= g.w;
+            for (int i = 0; i < OWN; ++i) {
+                const int t = (lr * OWN + i) / CT, j = (lr * OWN + i) % CT;
+                if (base + t < len && col + j < e)
+                    p.o[(size_t)(row0 + base + t) * p.heads * e + (size_t)h * e + col + j] = acc[i];
+            }
+        }
+        // S = diag(G_end) S_0 + KE^T U
 #pragma unroll
-            for (int s = 0; s < RC; ++s) {
-                const float4 k = *reinterpret_cast<const float4*>(KE + s * P + r0);
+        for (int u = 0; u < RUNS; ++u) {
+            const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(GE + r0 + RUN_STEP * u);
+#pragma unroll
+            for (int j = 0; j < CT; ++j) {
+                S[2 * u][j] = rc_mul2(S[2 * u][j], g.x);
+                S[2 * u + 1][j] = rc_mul2(S[2 * u + 1][j], g.y);
+            }
+        }
+#pragma unroll
+        for (int s = 0; s < RC; ++s) {
+            float uv[CT];
+            if constexpr (CT == 4) {
                 const float4 u4 = *reinterpret_cast<const float4*>(Us + s * CP + c0);
-                const float u[4] = { u4.x, u4.y, u4.z, u4.w };
+                uv[0] = u4.x, uv[1] = u4.y, uv[2] = u4.z, uv[3] = u4.w;
+            } else if constexpr (CT == 2) {
+                const float2 u2 = *reinterpret_cast<const float2*>(Us + s * CP + c0);
+                uv[0] = u2.x, uv[1] = u2.y;
+            } else {
+                uv[0] = Us[s * CP + c0];
+            }
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    S[j][0] = fmaf(k.x, u[j], S[j][0]);
-                    S[j][1] = fmaf(k.y, u[j], S[j][1]);
-                    S[j][2] = fmaf(k.z, u[j], S[j][2]);
-                    S[j][3] = fmaf(k.w, u[j], S[j][3]);
+            for (int u = 0; u < RUNS; ++u) {
+                const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(KE + s * DP + r0 + RUN_STEP * u);
+#pragma unroll
+                for (int j = 0; j < CT; ++j) {
+                    const uint64_t both = rc_pair(uv[j], uv[j]);
+                    S[2 * u][j] = rc_fma2(k.x, both, S[2 * u][j]);
+                    S[2 * u + 1][j] = rc_fma2(k.y, both, S[2 * u + 1][j]);
                 }
             }
-            // (nobody reads the copy between the first phase's barrier and the next chunk's)
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                *reinterpret_cast<float4*>(Sc + (c0 + j) * P + r0) = make_float4(S[j][0], S[j][1], S[j][2], S[j][3]);
         }
     }
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < RT / 2; ++i) {
+        const int r = r0 + RUN_STEP * (i / 2) + 2 * (i % 2);
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            if (r0 + i < d && col0 + c0 + j < e)
-                st[(size_t)(r0 + i) * e + col0 + c0 + j] = S[j][i];
+        for (int j = 0; j < CT; ++j) {
+            const float2 halves = rc_halves(S[i][j]);
+            if (r < d && col + j < e)
+                st[(size_t)r * e + col + j] = halves.x;
+            if (r + 1 < d && col + j < e)
+                st[(size_t)(r + 1) * e + col + j] = halves.y;
+        }
+    }
 }
 
 // ---------------------------------------------------------------- few tokens a sequence
@@ -477,7 +646,7 @@ recurrence_tokens_kernel(const RecurrenceParams p)
         const TX* k = static_cast<const TX*>(p.k) + row * p.stride + kh * d;
         float v = col < e ? to_f32(static_cast<const TX*>(p.v)[row * p.stride + (size_t)h * e + col]) : 0.f;
         if (p.activate)
-            v = lr_silu(v);
+            v = lr_silu<TX>(v);
         float beta = 1.f, ik = 1.f, iq = 1.f;
         if (DELTA) {
             beta = 1.f / (1.f + expf(-to_f32(static_cast<const TX*>(p.beta)[row * p.beta_stride + h])));
@@ -498,10 +667,10 @@ recurrence_tokens_kernel(const RecurrenceParams p)
                 kv = to_f32(k[c]);
                 qv = to_f32(q[c]);
                 if (p.activate)
-                    kv = lr_silu(kv), qv = lr_silu(qv);
+                    kv = lr_silu<TX>(kv), qv = lr_silu<TX>(qv);
                 kv *= ik;
                 qv *= iq;
-                g = DELTA ? expf(rate * lr_softplus(p.logits[row * p.logit_stride + h * d + c] + p.dt_bias[h * d + c])) : decay;
+                g = DELTA ? lr_decay<TX>(rate, p.logits[row * p.logit_stride + h * d + c] + p.dt_bias[h * d + c]) : decay;
             }
             vec[warp][0][i] = kv;
             vec[warp][1][i] = qv;
@@ -559,30 +728,34 @@ static inline int recurrence_sm_count()
     return sms;
 }
 
-template <int DP, int COLS, bool DELTA, typename TX>
+template <int DP, int RT, int CT, int COLS, bool DELTA, typename TX>
 static void launch_chunks(const RecurrenceParams& p, int seqs, cudaStream_t stream)
 {
-    const size_t smem = (size_t)(2 * rc_block(DP, DELTA) + COLS * rc_pitch(DP, DELTA) + 3 * RC * (COLS + 4)) * sizeof(float);
-    auto kernel = chunk_recurrence_kernel<DP, COLS, DELTA, TX>;
+    const size_t smem = (size_t)(2 * rc_block(DP, DELTA) + RC * (COLS + 4)) * sizeof(float);
+    auto kernel = chunk_recurrence_kernel<DP, RT, CT, COLS, DELTA, TX>;
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    launch(kernel, dim3((unsigned)((p.e + COLS - 1) / COLS), (unsigned)p.heads, (unsigned)seqs), dim3(DP * COLS / 16), smem,
-           stream, p);
+    launch(kernel, dim3((unsigned)((p.e + COLS - 1) / COLS), (unsigned)p.heads, (unsigned)seqs),
+           dim3((DP / RT) * (COLS / CT)), smem, stream, p);
 }
 
 template <int DP, bool DELTA, typename TX>
 static void launch_prompt(const RecurrenceParams& p, int seqs, int max_q_len, cudaStream_t stream)
 {
-    const size_t smem = (size_t)(DELTA ? 3 : 2) * RC * DP * sizeof(float);
+    const size_t smem = (size_t)(DELTA ? 3 * RC + 4 : 2 * RC) * DP * sizeof(float);
     auto prepare = recurrence_prepare_kernel<DP, DELTA, TX>;
     if (smem > 44 * 1024)
         cudaFuncSetAttribute(prepare, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch(prepare, dim3((unsigned)((max_q_len + RC - 1) / RC), (unsigned)p.heads, (unsigned)seqs), dim3(256), smem, stream, p);
-    // blocks of 32 columns where they give two SMs of three one, else of 16 (the work of a thread is the same)
-    if ((long long)((p.e + 31) / 32) * p.heads * seqs * 3 >= 2 * recurrence_sm_count())
-        launch_chunks<DP, 32, DELTA, TX>(p, seqs, stream);
+    // as few columns a block as give every SM one block and no more, and the fewer the smaller a thread's piece
+    constexpr int RT = DP >= 128 ? 8 : 4;
+    const long long per_head = (long long)p.heads * seqs, sms = recurrence_sm_count();
+    if (((p.e + 7) / 8) * per_head <= sms)
+        launch_chunks<DP, RT, DP >= 256 ? 2 : 1, 8, DELTA, TX>(p, seqs, stream);
+    else if (((p.e + 15) / 16) * per_head <= sms)
+        launch_chunks<DP, DP >= 256 ? 8 : 4, DP >= 128 ? 4 : 2, 16, DELTA, TX>(p, seqs, stream);
     else
-        launch_chunks<DP, 16, DELTA, TX>(p, seqs, stream);
+        launch_chunks<DP, RT, 4, 32, DELTA, TX>(p, seqs, stream);
 }
 
 template <bool DELTA, typename TX>

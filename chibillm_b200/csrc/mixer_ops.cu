@@ -160,7 +160,7 @@ latent_prepare_kernel(const TX* __restrict__ proj, long long stride, TX* __restr
 }
 
 // ---------------------------------------------------------------- q | k | v: biases, whole norm, append
-// One block per token; shared memory holds q | k with their biases in 32-bit.
+// One block per token; shared memory holds q | k with their biases in 32-bit, then the token's cosines and sines.
 template <typename TX, typename TC>
 __global__ void __launch_bounds__(512)
 qkv_bias_norm_append_kernel(const TX* __restrict__ proj, long long stride, TX* __restrict__ q_out,
@@ -204,10 +204,17 @@ qkv_bias_norm_append_kernel(const TX* __restrict__ proj, long long stride, TX* _
         // k follows q in the buffer and both have heads of d features: head h starts at h * d
         const int half = rot >> 1;
         const int heads = nq + (append ? nkv : 0);
-        for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
-            const int h = i / half, j = i - h * half;
+        float* angles = buf + (size_t)heads * d;           // cosines, then sines: once per token, not per head
+        for (int j = threadIdx.x; j < half; j += blockDim.x) {
             float sn, cs;
             sincosf((float)pos * inv_freq[j], &sn, &cs);
+            angles[j] = cs;
+            angles[half + j] = sn;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
+            const int h = i / half, j = i - h * half;
+            const float cs = angles[j], sn = angles[half + j];
             float* p = buf + (size_t)h * d;
             const float u = p[j], v = p[j + half];
             p[j] = u * cs - v * sn;
@@ -672,7 +679,7 @@ CHIBI_API int chibi_qkv_bias_norm_append(const void* proj, int x_type, long long
         return CHIBI_ERR_ARGUMENT;
     if (append && (!v_cache || !seq_of_token || !block_table || page_size <= 0))
         return CHIBI_ERR_ARGUMENT;
-    const size_t smem = (size_t)(nq + (append ? nkv : 0)) * d * sizeof(float);
+    const size_t smem = ((size_t)(nq + (append ? nkv : 0)) * d + rot) * sizeof(float);
     if (smem > 200 * 1024)
         return CHIBI_ERR_UNSUPPORTED;
     CHIBI_DISPATCH_TYPE(x_type, TX, CHIBI_DISPATCH_TYPE(cache_type, TC, {

@@ -167,6 +167,86 @@ short_conv_wide_kernel(const TX* __restrict__ x, long long x_stride, const float
     }
 }
 
+// The same for two to four taps, each input fetched once: a thread walks over its tokens with the last
+// TAPS - 1 inputs and all weights of its channels in registers.
+// SILU: silu of the sums (an activation named at run time would put every activation's code into each of the
+// unrolled elements: too much for the instruction cache, 68 us became 35).
+template <int TAPS, bool SILU, typename TX>
+__global__ void __launch_bounds__(128)
+short_conv_window_kernel(const TX* __restrict__ x, long long x_stride, const float* __restrict__ wt, TX* history,
+                         TX* __restrict__ out, long long out_stride, const int* __restrict__ q_start,
+                         const int* __restrict__ slots, int channels, int chunk, const float* __restrict__ bias,
+                         int add_input)
+{
+    pdl_enter();
+    constexpr int N = Pack<TX>::N, KEEP = TAPS - 1, AHEAD = 4;
+    const int ch = (blockIdx.x * blockDim.x + threadIdx.x) * N;
+    const int seq = blockIdx.z;
+    const int row0 = q_start[seq];
+    const int q_len = q_start[seq + 1] - row0;
+    const int first = blockIdx.y * chunk;
+    if (ch >= channels || first >= q_len)
+        return;
+    const int last = min(first + chunk, q_len);
+    TX* hist = history + (size_t)slots[seq] * KEEP * channels;
+    const TX* xc = x + (size_t)row0 * x_stride + ch;
+    auto input = [&](int m) {                              // input m of the step, or of the history before it
+        return m >= 0 ? xc + (size_t)m * x_stride : hist + (size_t)(KEEP + m) * channels + ch;
+    };
+    float w[TAPS][N], b[N], past[KEEP][N];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < N; e += 4)
+            Pack<float>::load(wt + (size_t)j * channels + ch + e, *reinterpret_cast<float(*)[4]>(&w[j][e]));
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+        b[e] = bias ? bias[ch + e] : 0.f;
+        if (add_input)
+            w[KEEP][e] += 1.f;                             // the token's own input is added
+    }
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+        Pack<TX>::load(input(first - KEEP + j), past[j]);
+    for (int i0 = first; i0 < last; i0 += AHEAD) {
+        float v[AHEAD][N];
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u)
+            if (i0 + u < last)
+                Pack<TX>::load(xc + (size_t)(i0 + u) * x_stride, v[u]);
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u) {
+            if (i0 + u >= last)
+                break;
+            float y[N];
+#pragma unroll
+            for (int e = 0; e < N; ++e) {
+                y[e] = b[e];
+#pragma unroll
+                for (int j = 0; j < KEEP; ++j)
+                    y[e] = fmaf(w[j][e], past[j][e], y[e]);
+                y[e] = fmaf(w[KEEP][e], v[u][e], y[e]);
+                if constexpr (SILU)
+                    y[e] = sizeof(TX) == 2 ? activate_rounded(y[e], 2) : activate(y[e], 2);
+#pragma unroll
+                for (int j = 0; j + 1 < KEEP; ++j)
+                    past[j][e] = past[j + 1][e];
+                past[KEEP - 1][e] = v[u][e];
+            }
+            Pack<TX>::store(out + (size_t)(row0 + i0 + u) * out_stride + ch, y);
+        }
+    }
+    if (first == 0) {
+        // (this thread alone reads the history: in its window above, before this)
+        for (int m = 0; m < KEEP; ++m) {
+            const int at = q_len + m;
+            float v[N];
+            Pack<TX>::load(at < KEEP ? hist + (size_t)at * channels + ch : xc + (size_t)(at - KEEP) * x_stride, v);
+            Pack<TX>::store(hist + (size_t)m * channels + ch, v);
+        }
+    }
+}
+
 // ---------------------------------------------------------------- delta rule
 constexpr int DELTA_LANES = 8;        // threads that share a value column (its key rows in equal parts)
 constexpr int DELTA_WARPS = 4;        // warps that run the recurrence
@@ -640,6 +720,21 @@ CHIBI_API int chibi_causal_conv(const void* x, int x_type, long long x_stride, c
              | reinterpret_cast<uintptr_t>(wt)) & 15) == 0;
     if (wide) {
         const int threads = channels / per;
+        if (taps >= 2 && taps <= 4 && (act < 0 || act == 2)) {
+            const int run = 8;                             // tokens a thread
+            const dim3 wgrid((unsigned)((threads + 127) / 128), (unsigned)((max_q_len + run - 1) / run), (unsigned)seqs);
+            CHIBI_DISPATCH_TYPE(x_type, TX, {
+                auto silu = taps == 2 ? short_conv_window_kernel<2, true, TX>
+                                      : taps == 3 ? short_conv_window_kernel<3, true, TX> : short_conv_window_kernel<4, true, TX>;
+                auto plain = taps == 2 ? short_conv_window_kernel<2, false, TX>
+                                       : taps == 3 ? short_conv_window_kernel<3, false, TX>
+                                                   : short_conv_window_kernel<4, false, TX>;
+                auto kernel = act == 2 ? silu : plain;
+                launch(kernel, wgrid, dim3(128), 0, stream, (const TX*)x, x_stride, wt, (TX*)history, (TX*)out, out_stride,
+                       q_start, slots, channels, run, bias, add_input);
+            });
+            return launch_status();
+        }
         const dim3 grid((unsigned)((threads + 127) / 128), (unsigned)chunks, (unsigned)seqs);
         CHIBI_DISPATCH_TYPE(x_type, TX, {
             launch(short_conv_wide_kernel<TX>, grid, dim3(128), 0, stream, (const TX*)x, x_stride, wt, (TX*)history,

@@ -17,6 +17,18 @@ namespace chibi {
 
 using namespace sm100;
 
+__device__ __forceinline__ void store4(float* dst, float a, float b, float c, float d)
+{
+    *reinterpret_cast<float4*>(dst) = make_float4(a, b, c, d);
+}
+__device__ __forceinline__ void store4(__nv_bfloat16* dst, float a, float b, float c, float d)
+{
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a, b), hi = __floats2bfloat162_rn(c, d);
+    uint2 v;
+    v.x = *reinterpret_cast<const uint32_t*>(&lo), v.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = v;
+}
+
 struct SublayerEnd {
     float* residual;                 // [rows, n]
     const float* delta;              // [splits, rows, n]
@@ -33,17 +45,19 @@ struct SublayerEnd {
     int n;
 };
 
-// A thread owns four neighbouring columns of a row (n / 4 = gridDim.x * blockDim.x); the gridDim.x CTAs of a
-// row form a cluster that adds up its sums of squares through one another's shared memory.
-template <typename TW, typename TO>
-__global__ void __launch_bounds__(1024)
+// A thread owns V runs of four neighbouring columns of a row (n = 4 V gridDim.x blockDim.x), a run's threads side
+// by side; the gridDim.x CTAs of a row form a cluster that adds up its sums of squares through one another's
+// shared memory.  Everything a row needs is asked for before its first sum of squares: the earlier results'
+// weighted sum does not depend on this layer's.
+template <int V, typename TW, typename TO>
+__global__ void __launch_bounds__(1024 / V)
 sublayer_end_kernel(const SublayerEnd p, const TW* __restrict__ norm_w, TO* __restrict__ out)
 {
     pdl_trigger();
     __shared__ float scratch[33];
     __shared__ float sums[2][8];
     const int parts = gridDim.x;
-    const int c = 4 * (blockIdx.x * blockDim.x + threadIdx.x);
+    const int c = 4 * (blockIdx.x * V * blockDim.x + threadIdx.x), step = 4 * blockDim.x;
     const long long t = blockIdx.y + (long long)blockIdx.z * gridDim.y;
     if (t >= p.rows)
         return;                                        // a whole cluster leaves together
@@ -61,74 +75,94 @@ sublayer_end_kernel(const SublayerEnd p, const TW* __restrict__ norm_w, TO* __re
             total += sums[which][r];
         return total;
     };
-    // weights are not written while a step runs: fetched before the kernel ahead is through
-    const float4 v4 = *reinterpret_cast<const float4*>(p.vec + c);
-    float4 b4 = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (p.bias)
-        b4 = *reinterpret_cast<const float4*>(p.bias + c);
-    float w4[4] = { 0.f, 0.f, 0.f, 0.f };
-    if (out) {
-#pragma unroll
-        for (int u = 0; u < 4; ++u)
-            w4[u] = to_f32(norm_w[c + u]) + p.offset;
-    }
+    auto load4 = [](const float* src) { return *reinterpret_cast<const float4*>(src); };
     if (parts > 1)
         cluster_sync();                                // every CTA of the row has started: its shared memory is there
     pdl_wait();
-    float4 r = *reinterpret_cast<const float4*>(p.residual + at);
-    float4 y = b4;
-    for (int s0 = 0; s0 < p.splits; s0 += 8) {
-        float4 q[8];
+    float4 r[V], y[V], sum[V];
+    float own = 1.f;
 #pragma unroll
-        for (int u = 0; u < 8; ++u)
-            q[u] = s0 + u < p.splits ? *reinterpret_cast<const float4*>(p.delta + (size_t)(s0 + u) * plane + at)
-                                     : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < V; ++i) {
+        r[i] = load4(p.residual + at + i * step);
+        y[i] = p.bias ? load4(p.bias + c + i * step) : make_float4(0.f, 0.f, 0.f, 0.f);
+        sum[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    constexpr int AHEAD = V == 1 ? 8 : 2;              // arrays whose loads are in flight together
+    for (int s0 = 0; s0 < p.splits; s0 += AHEAD) {
+        float4 q[AHEAD][V];
 #pragma unroll
-        for (int u = 0; u < 8; ++u)
-            y.x += q[u].x, y.y += q[u].y, y.z += q[u].z, y.w += q[u].w;
+        for (int u = 0; u < AHEAD; ++u)
+#pragma unroll
+            for (int i = 0; i < V; ++i)
+                q[u][i] = s0 + u < p.splits ? load4(p.delta + (size_t)(s0 + u) * plane + at + i * step)
+                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u)
+#pragma unroll
+            for (int i = 0; i < V; ++i)
+                y[i].x += q[u][i].x, y[i].y += q[u][i].y, y[i].z += q[u][i].z, y[i].w += q[u][i].w;
+    }
+    if (p.outputs) {
+        own = p.weights[p.earlier];
+        for (int j0 = 0; j0 < p.earlier; j0 += AHEAD) {
+            float4 q[AHEAD][V];
+            float k[AHEAD];
+#pragma unroll
+            for (int u = 0; u < AHEAD; ++u) {
+                const bool on = j0 + u < p.earlier;
+                k[u] = on ? p.weights[j0 + u] : 0.f;
+#pragma unroll
+                for (int i = 0; i < V; ++i)
+                    q[u][i] = on ? load4(p.outputs + (size_t)(j0 + u) * plane + at + i * step)
+                                 : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int u = 0; u < AHEAD; ++u)
+#pragma unroll
+                for (int i = 0; i < V; ++i) {
+                    sum[i].x = fmaf(k[u], q[u][i].x, sum[i].x);
+                    sum[i].y = fmaf(k[u], q[u][i].y, sum[i].y);
+                    sum[i].z = fmaf(k[u], q[u][i].z, sum[i].z);
+                    sum[i].w = fmaf(k[u], q[u][i].w, sum[i].w);
+                }
+        }
     }
     float inv = 1.f;
     if (p.y_eps >= 0.f) {
-        const float s = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w)));
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < V; ++i)
+            s = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, s))));
         inv = 1.f / sqrtf(whole_row(s, 0) / (float)p.n + p.y_eps);
     }
-    r.x = fmaf(v4.x, y.x * inv, r.x);
-    r.y = fmaf(v4.y, y.y * inv, r.y);
-    r.z = fmaf(v4.z, y.z * inv, r.z);
-    r.w = fmaf(v4.w, y.w * inv, r.w);
-    if (p.outputs) {
-        if (p.keep)
-            *reinterpret_cast<float4*>(p.outputs + (size_t)p.earlier * plane + at) = r;
-        const float own = p.weights[p.earlier];
-        r.x *= own, r.y *= own, r.z *= own, r.w *= own;
-        for (int j0 = 0; j0 < p.earlier; j0 += 4) {
-            float4 q[4];
-            float k[4];
+    float s = 0.f;
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                const bool on = j0 + u < p.earlier;
-                k[u] = on ? p.weights[j0 + u] : 0.f;
-                q[u] = on ? *reinterpret_cast<const float4*>(p.outputs + (size_t)(j0 + u) * plane + at)
-                          : make_float4(0.f, 0.f, 0.f, 0.f);
-            }
-#pragma unroll
-            for (int u = 0; u < 4; ++u) {
-                r.x = fmaf(k[u], q[u].x, r.x);
-                r.y = fmaf(k[u], q[u].y, r.y);
-                r.z = fmaf(k[u], q[u].z, r.z);
-                r.w = fmaf(k[u], q[u].w, r.w);
-            }
+    for (int i = 0; i < V; ++i) {
+        const float4 v = load4(p.vec + c + i * step);
+        r[i].x = fmaf(v.x, y[i].x * inv, r[i].x);
+        r[i].y = fmaf(v.y, y[i].y * inv, r[i].y);
+        r[i].z = fmaf(v.z, y[i].z * inv, r[i].z);
+        r[i].w = fmaf(v.w, y[i].w * inv, r[i].w);
+        if (p.outputs) {
+            if (p.keep)
+                *reinterpret_cast<float4*>(p.outputs + (size_t)p.earlier * plane + at + i * step) = r[i];
+            r[i].x = fmaf(own, r[i].x, sum[i].x);
+            r[i].y = fmaf(own, r[i].y, sum[i].y);
+            r[i].z = fmaf(own, r[i].z, sum[i].z);
+            r[i].w = fmaf(own, r[i].w, sum[i].w);
         }
+        *reinterpret_cast<float4*>(p.residual + at + i * step) = r[i];
+        s = fmaf(r[i].x, r[i].x, fmaf(r[i].y, r[i].y, fmaf(r[i].z, r[i].z, fmaf(r[i].w, r[i].w, s))));
     }
-    *reinterpret_cast<float4*>(p.residual + at) = r;
     if (!out)
         return;
-    const float s = fmaf(r.x, r.x, fmaf(r.y, r.y, fmaf(r.z, r.z, r.w * r.w)));
     const float f = 1.f / sqrtf(whole_row(s, 1) / (float)p.n + p.eps);
-    out[at] = from_f32<TO>(r.x * f * w4[0]);
-    out[at + 1] = from_f32<TO>(r.y * f * w4[1]);
-    out[at + 2] = from_f32<TO>(r.z * f * w4[2]);
-    out[at + 3] = from_f32<TO>(r.w * f * w4[3]);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const TW* w = norm_w + c + i * step;
+        store4(out + at + i * step, r[i].x * f * (to_f32(w[0]) + p.offset), r[i].y * f * (to_f32(w[1]) + p.offset),
+               r[i].z * f * (to_f32(w[2]) + p.offset), r[i].w * f * (to_f32(w[3]) + p.offset));
+    }
 }
 
 // The same for any width: one block per row, the row in shared memory.
@@ -224,6 +258,16 @@ __device__ __forceinline__ float xielu(float z, float pos, float neg)
     return z > 0.f ? fmaf(pos * z, z, 0.5f * z) : fmaf(neg, expm1f(z) - z, 0.5f * z);
 }
 
+// The same for results that become bfloat16 at once: exp(z) - 1 - z as the first terms of its series next to
+// zero (where the difference would cancel) and as the difference of the faster exponential elsewhere; good to
+// 1e-4 of the result.
+__device__ __forceinline__ float xielu_rounded(float z, float pos, float neg)
+{
+    const float series = z * z * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f);
+    const float rest = z > -0.0625f ? series : __expf(z) - 1.f - z;
+    return z > 0.f ? fmaf(pos * z, z, 0.5f * z) : fmaf(neg, rest, 0.5f * z);
+}
+
 // x: [splits, rows, n] (partial sums of a product when there are several) or an array that may be `out`
 template <typename TX, typename TO>
 __global__ void bias_xielu_kernel(const TX* x, int splits, const float* __restrict__ bias, TO* out, long long rows, int n,
@@ -287,7 +331,8 @@ __global__ void bias_xielu_wide_kernel(const __nv_bfloat16* x, const float* __re
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 z = __bfloat1622float2(h[j]);
-            h[j] = __floats2bfloat162_rn(xielu(z.x + b[2 * j], pos, neg), xielu(z.y + b[2 * j + 1], pos, neg));
+            h[j] = __floats2bfloat162_rn(xielu_rounded(z.x + b[2 * j], pos, neg),
+                                         xielu_rounded(z.y + b[2 * j + 1], pos, neg));
         }
         *reinterpret_cast<uint4*>(out + t * n + c) = raw;
     }
@@ -318,26 +363,33 @@ CHIBI_API int chibi_sublayer_end(float* residual, const float* delta, int splits
                           | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(vec)
                           | reinterpret_cast<uintptr_t>(outputs);
     const int n4 = n / 4;
-    int parts = 0;                     // CTAs per row: many for few rows, else as few as the block size allows
-    if (n % 128 == 0 && (all & 15) == 0) {
-        for (int cand = 1; cand <= 8; ++cand) {
-            if (n4 % cand != 0 || (n4 / cand) % 32 != 0 || n4 / cand > 1024)
-                continue;
-            parts = cand;
-            if (rows > 64)
-                break;
+    int parts = 0, runs = 1;           // CTAs per row and runs of columns per thread
+    if (n % 128 == 0 && (all & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
+        if (rows <= 64) {
+            // few rows: as many CTAs to a row as divide it evenly
+            for (int cand = 1; cand <= 8; ++cand)
+                if (n4 % cand == 0 && (n4 / cand) % 32 == 0 && n4 / cand <= 1024)
+                    parts = cand;
+        } else {
+            // many rows: small blocks, several of them to an SM
+            runs = n4 % 128 == 0 && n4 >= 512 ? 4 : (n4 % 64 == 0 && n4 >= 256 ? 2 : 1);
+            for (int cand = 1; cand <= 8 && parts == 0; ++cand)
+                if (n4 % (runs * cand) == 0 && (n4 / (runs * cand)) % 32 == 0 && n4 / (runs * cand) <= 1024 / runs)
+                    parts = cand;
         }
     }
     if (parts > 0) {
         const unsigned gy = (unsigned)(rows < 32768 ? rows : 32768), gz = (unsigned)((rows + gy - 1) / gy);
         if (gz > 65535)
             return CHIBI_ERR_UNSUPPORTED;
-        const dim3 grid((unsigned)parts, gy, gz), block((unsigned)(n4 / parts));
+        const dim3 grid((unsigned)parts, gy, gz), block((unsigned)(n4 / (parts * runs)));
         CHIBI_DISPATCH_TYPE(w_type, TW, CHIBI_DISPATCH_TYPE(out_type, TO, {
+            auto kernel = runs == 4 ? sublayer_end_kernel<4, TW, TO>
+                                    : runs == 2 ? sublayer_end_kernel<2, TW, TO> : sublayer_end_kernel<1, TW, TO>;
             if (parts > 1)
-                launch_cluster_x(sublayer_end_kernel<TW, TO>, grid, block, 0, stream, parts, p, (const TW*)norm_w, (TO*)out);
+                launch_cluster_x(kernel, grid, block, 0, stream, parts, p, (const TW*)norm_w, (TO*)out);
             else
-                launch(sublayer_end_kernel<TW, TO>, grid, block, 0, stream, p, (const TW*)norm_w, (TO*)out);
+                launch(kernel, grid, block, 0, stream, p, (const TW*)norm_w, (TO*)out);
         }));
         return launch_status();
     }

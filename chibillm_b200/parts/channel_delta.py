@@ -28,6 +28,11 @@ def _round8(n: int) -> int:
     return (n + 7) // 8 * 8
 
 
+def _whole_tiles(n: int) -> int:
+    """The stacked product's rows: a large one in whole tiles of 256 (rows of zeros fill the last)."""
+    return (n + 255) // 256 * 256 if n >= 2048 else _round8(n)
+
+
 class ChannelDelta(Mixer):
     can_overwrite = True
     accepts_scaled_rows = True       # x goes to the stacked product and nowhere else
@@ -75,7 +80,7 @@ class ChannelDelta(Mixer):
         t = {role: tensors[name] for role, name in self.names.items() if name in tensors}
         first = t["q_proj"]
         ra, rg = s.decay_rank, s.gate_rank
-        stacked = torch.zeros((_round8(self.beta_at + s.num_heads), s.hidden_size), dtype=first.dtype, device=first.device)
+        stacked = torch.zeros((_whole_tiles(self.beta_at + s.num_heads), s.hidden_size), dtype=first.dtype, device=first.device)
         at = 0
         for role in ("q_proj", "k_proj", "v_proj"):
             stacked[at:at + t[role].shape[0]] = t[role]
