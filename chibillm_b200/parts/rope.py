@@ -90,6 +90,10 @@ class RotaryEncoding(PositionEncoding):
                 raise ValueError("a stretched rotation needs positive factor, original positions and turn counts")
             self.inv_freq = stretched_inverse_frequencies(spec).to(runtime.device)
             self.amplitude = float(spec.amplitude_slope) * math.log(float(spec.scaling_factor)) + 1.0
+        elif spec.interleaved:
+            # made in 64-bit and rounded once
+            j = torch.arange(spec.rotary_dim // 2, dtype=torch.float64)
+            self.inv_freq = (float(spec.theta) ** (-2.0 * j / spec.rotary_dim)).to(torch.float32).to(runtime.device)
         else:
             self.inv_freq = rotary_inverse_frequencies(spec.theta, spec.rotary_dim).to(runtime.device)
 
@@ -112,7 +116,8 @@ class RotaryEncoding(PositionEncoding):
             return None                      # the table's readers rotate with amplitude one
         s = self.spec
         key = ("rope", float(s.theta), int(s.rotary_dim), float(s.scaling_factor), int(s.original_positions),
-               float(s.fast_turns), float(s.slow_turns), tuple(getattr(s, "wavelength_bands", None) or ()))
+               float(s.fast_turns), float(s.slow_turns), tuple(getattr(s, "wavelength_bands", None) or ()),
+               bool(s.interleaved))
         table = ctx.shared.get(key)
         if table is None:
             table = ctx.workspace.get("rope.table." + ".".join(str(v) for v in key[1:]),
