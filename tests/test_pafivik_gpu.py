@@ -615,6 +615,19 @@ def test_cutting_and_batching(folders, expected, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_sublayers_that_add_into_a_zeroed_array(folders, expected, dtype, monkeypatch):
+    """The same model with every part adding its result instead of writing it."""
+    from chibillm_b200.parts import attention, channel_delta, linear_attention, mlp
+    reqs, ref, margins = expected["P3", dtype][:3]
+    for part in (attention.PagedAttention, channel_delta.ChannelDelta, linear_attention.LinearAttention, mlp.DenseMLP,
+                 mlp.RoutedExperts):
+        monkeypatch.setattr(part, "can_overwrite", False)
+    runner = make_runner(folders["P3", dtype], dtype, 16, 192)
+    compare(helpers.run_trace(runner, helpers.trace_last_decoded(reqs, 20)), ref, margins, dtype,
+            f"pafivik P3 {dtype}, sublayers added")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_a_batch_against_each_request_alone(folders, dtype):
     """Four unequal requests in the same steps against each in steps of its own, both against the plain
     implementation."""

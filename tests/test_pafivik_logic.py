@@ -228,6 +228,21 @@ def test_each_options_weight_is_read(tmp_path):
         assert float((got - want).abs().max()) < 1e-4 * float(want.abs().max()), name
 
 
+def test_sublayers_that_add_into_a_zeroed_array(tmp_path, monkeypatch):
+    """The same model with every part adding its result instead of writing it (what a part without
+    ``can_overwrite`` does): the bias of the dense feed-forward then joins through the part itself."""
+    from chibillm_b200.parts import attention, channel_delta, linear_attention, mlp
+    cfg = pafivik_models.get("P1")
+    folder = pafivik_models.write_model(cfg, str(tmp_path / "p1"), seed=13)
+    reqs = helpers.random_requests(cfg["vocab"], [33], seed=3)
+    ref = pafivik_models.plain_logits(cfg, 13, reqs)
+    for part in (attention.PagedAttention, channel_delta.ChannelDelta, linear_attention.LinearAttention, mlp.DenseMLP,
+                 mlp.RoutedExperts):
+        monkeypatch.setattr(part, "can_overwrite", False)
+    got = helpers.run_trace(cpu_runner(folder, 4, 64), helpers.trace_portions(reqs, seed=2))
+    helpers.assert_logits_close(got, ref, helpers.TOL["float32"], "pafivik, sublayers added")
+
+
 def test_spec_combinations_that_are_refused():
     from dataclasses import replace
     from chibillm_b200.config import PafivikConfig
