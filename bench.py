@@ -15,8 +15,8 @@ its time, against the measured copy bandwidth; ``points`` decode at batch 1 and
 filled by real prefill steps for the end-to-end run and with random values for
 the device-timed runs (the work of a decode step does not depend on the values).
 
-``--design gitipel`` (or ``fokurax``, ``pitudra``, ``dogetar``, ``pafivik``) prints, instead of the record, prefill
-and decode of that design beside Qwen3 (Pitudra: beside Fokurax, Dogetar: beside Pitudra, Pafivik: beside Gitipel) at
+``--design gitipel`` (or ``fokurax``, ``pitudra``, ``dogetar``, ``pafivik``, ``lefavik``) prints, instead of the record, prefill
+and decode of that design beside Qwen3 (Pitudra: beside Fokurax, Dogetar: beside Pitudra, Pafivik: beside Gitipel, Lefavik: beside Pitudra) at
 equal layer sizes, with the time of every kernel.
 
 ``--timeline`` prints, instead of the record, when the CTAs of every kernel of one
@@ -499,6 +499,29 @@ def pafivik_config(width, heads, kv_heads, dim, ff, vocab=32768):
             "layers": [delta(dense), delta(experts), attention(dense), lightning, delta(dense), attention(experts)]}
 
 
+def lefavik_config(width, heads, kv_heads, dim, ff, vocab=32768):
+    """Six layers, each with its two sublayers side by side under one norm and a dense feed-forward: latent
+    attention (a latent of 192 numbers and a rotated part of 64, 96 and 32 with heads of 64; queries straight
+    from the layer's input), attention in a window of 1,024 positions with a distance bias, and latent attention
+    on the first layer's cache; twice over, the second group's reader on the second group's cache."""
+    rot = dim // 2
+    dense = {"kind": "dense", "ff": ff}
+
+    def latent(kv_from=None):
+        m = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": dim, "kv_rank": 3 * rot,
+             "rot": {"base": 1e6, "dims": rot}, "scale": (dim + rot) ** -0.5}
+        if kv_from is not None:
+            m["kv_from"] = kv_from
+        return {"type": "latent_attention", "mixer": m, "mlp": dense}
+
+    window = {"type": "attention", "mlp": dense,
+              "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                        "mask": {"size": 1024}, "q_temp": {"coef": 0.2, "every": 512}}}
+    return {"architecture": "Lefavik", "vocab": vocab, "width": width, "max_positions": 8192, "norm": {"eps": 1e-5},
+            "embedding": {"scale": width ** 0.5}, "logit_scale": 0.5,
+            "layers": [latent(), window, latent(0), latent(), window, latent(3)]}
+
+
 def qwen3_config_like(width, heads, kv_heads, dim, ff, layers=6, vocab=32768):
     cfg = dict(QWEN3_8B)
     cfg.update(num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads, num_key_value_heads=kv_heads,
@@ -569,11 +592,12 @@ def compare_designs(sizes, prompt_tokens, batch, held, steps, warmup, design="gi
     """Another design beside Qwen3 at equal layer sizes (six layer runs each, random weights);
     Pitudra beside Fokurax, the design nearest to it (routed experts, layers that read another
     layer's cache, a token input per layer); Dogetar beside Pitudra (a recurrent state, routed experts,
-    windows, sinks and gates); Pafivik beside Gitipel (a delta rule beside attention)."""
+    windows, sinks and gates); Pafivik beside Gitipel (a delta rule beside attention); Lefavik beside Pitudra
+    (attention over cached latents, layers that read another layer's cache)."""
     make = {"gitipel": gitipel_config, "fokurax": fokurax_config, "pitudra": pitudra_config,
-            "dogetar": dogetar_config, "pafivik": pafivik_config}[design]
+            "dogetar": dogetar_config, "pafivik": pafivik_config, "lefavik": lefavik_config}[design]
     beside, make_other = {"pitudra": ("fokurax", fokurax_config), "dogetar": ("pitudra", pitudra_config),
-                          "pafivik": ("gitipel", gitipel_config)}.get(design, ("qwen3", qwen3_config_like))
+                          "pafivik": ("gitipel", gitipel_config), "lefavik": ("pitudra", pitudra_config)}.get(design, ("qwen3", qwen3_config_like))
     result = {"metric": f"prefill and decode of {design.capitalize()} beside {beside.capitalize()} at equal layer sizes",
               "layer_runs": 6,
               "prompt_tokens": prompt_tokens, "decode_batch": batch, "decode_tokens_held": held, "dtype": "bf16",
@@ -666,9 +690,9 @@ def main() -> int:
     ap.add_argument("--check-tokens", type=int, default=0,
                     help="with --mixed-requests: also generate this many tokens of every request with the 32-bit "
                          "engine under two budgets and report how the runs agree")
-    ap.add_argument("--design", default=None, choices=["gitipel", "fokurax", "pitudra", "dogetar", "pafivik"],
+    ap.add_argument("--design", default=None, choices=["gitipel", "fokurax", "pitudra", "dogetar", "pafivik", "lefavik"],
                     help="instead of the record: prefill and decode of this design beside Qwen3 (pitudra: beside "
-                         "fokurax, dogetar: beside pitudra, pafivik: beside gitipel) at equal layer sizes "
+                         "fokurax, dogetar and lefavik: beside pitudra, pafivik: beside gitipel) at equal layer sizes "
                          "(--design-sizes), with the time of every kernel")
     ap.add_argument("--design-sizes", default="small,medium,large",
                     help="layer sizes for --design, with commas between them: " + ", ".join(DESIGN_SIZES))

@@ -27,6 +27,10 @@ from .pafivik import ARCHITECTURE as PAFIVIK_ARCHITECTURE, SHAPES_KEY as _PAFIVI
 
 register_architecture(PAFIVIK_ARCHITECTURE, PafivikConfig.from_dict, PafivikConfig.model_spec, replace=True,
                       shapes_key=_PAFIVIK_SHAPES)
+from .lefavik import ARCHITECTURE as LEFAVIK_ARCHITECTURE, SHAPES_KEY as _LEFAVIK_SHAPES, LefavikConfig
+
+register_architecture(LEFAVIK_ARCHITECTURE, LefavikConfig.from_dict, LefavikConfig.model_spec, replace=True,
+                      shapes_key=_LEFAVIK_SHAPES)
 
 __all__ = [
     "ConfigError", "KeyReader", "read_config_json",
@@ -34,7 +38,7 @@ __all__ = [
     "NormSpec", "PositionSpec", "RunStep", "DeltaRuleSpec", "DenseMLPSpec", "ShortConvSpec", "GitipelConfig",
     "TableExpertsSpec", "TokenInputSpec", "FokuraxConfig", "GatedRecurrenceSpec", "LatentAttentionSpec",
     "RoutedExpertsSpec", "PitudraConfig", "StateSpaceSpec", "ParallelMixersSpec", "DogetarConfig",
-    "ChannelDeltaSpec", "LinearAttentionSpec", "PafivikConfig",
+    "ChannelDeltaSpec", "LinearAttentionSpec", "PafivikConfig", "LefavikConfig",
     "Architecture", "find_architecture", "load_config", "register_architecture",
     "registered_architectures", "unregister_architecture", "Qwen3Config",
 ]

@@ -122,6 +122,9 @@ class AttentionSpec(MixerSpec):
     number per head (role "head_gate", [num_heads, hidden]), before the output projection.
     ``biases`` together with ``qk_norm``: the biases are added first, then every q and k head is
     normalised with the shared weight, then rotated.
+    ``sink_value`` (None: off): the same number joins every head's denominator as exp(sink_value), unscaled; no
+    tensor (0: the softmax with one added to its denominator).  ``query_temperature`` (c, every): the query at
+    position p, after its norm, is multiplied by 1 + c * ln(floor((p + 1) / every) + 1).
     """
 
     hidden_size: int = 0
@@ -149,6 +152,8 @@ class AttentionSpec(MixerSpec):
     differential: Optional[float] = None
     differential_eps: float = 0.0
     head_gate: bool = False
+    sink_value: Optional[float] = None
+    query_temperature: Optional[Tuple[float, int]] = None
 
 
 @dataclass(frozen=True)
@@ -205,6 +210,9 @@ class LatentAttentionSpec(MixerSpec):
     ``sink``, ``own_kv`` and ``cache_window`` as for AttentionSpec (a layer
     without W_dkv reads another step's cache with W_uk and W_uv of its own).
     ``position`` rotates the ``rope_dim`` part (its ``head_dim`` is ``rope_dim``).
+    ``q_rank`` 0: the queries have no latent of their own, q = W_q x (role "q_proj",
+    the same layout).  ``head_gate``: head h's output is multiplied by sigmoid(Wg x)[h]
+    before the output projection (role "head_gate", [num_heads, hidden]).
     """
 
     hidden_size: int = 0
@@ -221,6 +229,7 @@ class LatentAttentionSpec(MixerSpec):
     own_kv: bool = True
     position: PositionSpec = PositionSpec(kind="none")
     cache_window: object = "same"
+    head_gate: bool = False
 
 
 @dataclass(frozen=True)

@@ -42,8 +42,8 @@ struct GemmParams {
     const float* residual;
     long long res_stride;
     float* partial;        // [splits][M][N] when the K range is split through global memory, else null
-    int swiglu;            // the rows of w come in blocks of 64 gate rows then 64 up rows; out[M, N / 2] =
-                           // silu(gate) * up
+    int swiglu;            // 0: no; else the rows of w come in blocks of 64 gate rows then 64 up rows and
+                           // out[M, N / 2] = act(gate) * up, act: 1 silu, 2 the tanh form of gelu
     int act;               // 0: none; k > 0: activation k - 1 (see activate()) on the sums where they become
                            // the output's type (no residual with it)
     int* error;
@@ -88,6 +88,21 @@ struct GemmParams {
     int h_w_type, h_nq, h_nkv, h_page_size;
     float h_eps, h_offset;
 };
+
+// act(g) * u of a gated product (GemmParams::swiglu): g / (1 + exp(-z)) with z = g for silu and, since
+// (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y)), z = 2 sqrt(2 / pi) (g + 0.044715 g^3) for the tanh form of gelu.
+__device__ __forceinline__ float gate_argument(float g, int kind)
+{
+    return kind == 2 ? g * fmaf(1.59576912160573071f * 0.044715f, g * g, 1.59576912160573071f) : g;
+}
+__device__ __forceinline__ float gate_mul(float g, float u, int kind)
+{
+    return __fdividef(g, 1.f + __expf(-gate_argument(g, kind))) * u;
+}
+__device__ __forceinline__ float gate_mul_exact(float g, float u, int kind)
+{
+    return (g / (1.f + expf(-gate_argument(g, kind)))) * u;
+}
 
 template <int BN>
 struct GemmSmem {
@@ -256,7 +271,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                                 for (int q = 0; q < 4; ++q) {
                                     const float g0 = __uint_as_float(g[8 * j + 2 * q]), g1 = __uint_as_float(g[8 * j + 2 * q + 1]);
                                     const float u0 = __uint_as_float(u[8 * j + 2 * q]), u1 = __uint_as_float(u[8 * j + 2 * q + 1]);
-                                    h[q] = __floats2bfloat162_rn((g0 / (1.f + expf(-g0))) * u0, (g1 / (1.f + expf(-g1))) * u1);
+                                    h[q] = __floats2bfloat162_rn(gate_mul_exact(g0, u0, p.swiglu), gate_mul_exact(g1, u1, p.swiglu));
                                 }
                                 reinterpret_cast<uint4*>(dst)[j] = *reinterpret_cast<uint4*>(h);
                             }
@@ -264,7 +279,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a,
                             for (int j = 0; j < 32; ++j)
                                 if (feat0 + j < inter) {
                                     const float gv = __uint_as_float(g[j]), uv = __uint_as_float(u[j]);
-                                    dst[j] = __float2bfloat16_rn((gv / (1.f + expf(-gv))) * uv);
+                                    dst[j] = __float2bfloat16_rn(gate_mul_exact(gv, uv, p.swiglu));
                                 }
                         }
                     }
@@ -360,11 +375,6 @@ constexpr int EPILOGUE_STAGE_BYTES = 32 * 128;     // per epilogue warp
 __device__ __forceinline__ uint4* stage_unit(uint8_t* stage, int row, int unit)
 {
     return reinterpret_cast<uint4*>(stage + row * 128 + ((unit ^ (row & 7)) << 4));
-}
-
-__device__ __forceinline__ float silu_mul(float g, float u)
-{
-    return __fdividef(g, 1.f + __expf(-g)) * u;
 }
 
 // One 128-row tile of the q | k | v product as one or two heads (see GemmParams): this thread's token is
@@ -562,9 +572,10 @@ __device__ __forceinline__ void epilogue_token_rows(const GemmParams& p, uint32_
 #pragma unroll
                     for (int q = 0; q < 4; ++q)
                         v[q] = __floats2bfloat162_rn(
-                            silu_mul(inv * __uint_as_float(g[8 * j + 2 * q]), inv * __uint_as_float(u[8 * j + 2 * q])),
-                            silu_mul(inv * __uint_as_float(g[8 * j + 2 * q + 1]),
-                                     inv * __uint_as_float(u[8 * j + 2 * q + 1])));
+                            gate_mul(inv * __uint_as_float(g[8 * j + 2 * q]), inv * __uint_as_float(u[8 * j + 2 * q]),
+                                     p.swiglu),
+                            gate_mul(inv * __uint_as_float(g[8 * j + 2 * q + 1]),
+                                     inv * __uint_as_float(u[8 * j + 2 * q + 1]), p.swiglu));
                     *stage_unit(stage, lane, 4 * h + j) = *reinterpret_cast<uint4*>(v);
                 }
             }
@@ -598,7 +609,7 @@ __device__ __forceinline__ void epilogue_token_rows(const GemmParams& p, uint32_
                 for (int j = 0; j < 32; ++j)
                     if (feat0 + j < inter) {
                         const float gv = __uint_as_float(g[j]), uv = __uint_as_float(u[j]);
-                        dst[j] = __float2bfloat16_rn((gv / (1.f + expf(-gv))) * uv);
+                        dst[j] = __float2bfloat16_rn(gate_mul_exact(gv, uv, p.swiglu));
                     }
             }
             __syncwarp();
@@ -1724,7 +1735,8 @@ CHIBI_API int chibi_gemm_reset_stream_counters(cudaStream_t stream)
 
 // out = x * w^T of more than 64 rows with what follows it done in the same kernel: + residual, or
 // (epilogue 1) SwiGLU over w's rows arranged as blocks of 64 gate rows followed by their 64 up
-// rows (out is then [M, N / 2], bfloat16).  Few rows split their K range instead
+// rows (out is then [M, N / 2], bfloat16); epilogue 6: the same with the tanh form of gelu as the gate's
+// activation.  Few rows split their K range instead
 // (chibi_gemm_bf16_partial and the kernels that finish a split product).
 CHIBI_API int chibi_gemm_bf16_fused(const void* x, const void* w, void* out, int out_type,
                                     const float* residual, int M, int N, int K, long long x_stride,
@@ -1739,11 +1751,11 @@ CHIBI_API int chibi_gemm_bf16_fused(const void* x, const void* w, void* out, int
         return CHIBI_ERR_UNSUPPORTED;
     if (out_type != CHIBI_F32 && out_type != CHIBI_BF16)
         return CHIBI_ERR_ARGUMENT;
-    if (epilogue == 1 && (N % 128 != 0 || out_type != CHIBI_BF16 || residual))
+    if ((epilogue == 1 || epilogue == 6) && (N % 128 != 0 || out_type != CHIBI_BF16 || residual))
         return CHIBI_ERR_UNSUPPORTED;
-    if (epilogue < 0 || epilogue > 5)
+    if (epilogue < 0 || epilogue > 6)
         return CHIBI_ERR_ARGUMENT;
-    if (epilogue >= 2 && (out_type != CHIBI_BF16 || residual))
+    if (epilogue >= 2 && epilogue <= 5 && (out_type != CHIBI_BF16 || residual))
         return CHIBI_ERR_UNSUPPORTED;      // epilogue 2 .. 5: activation 0 .. 3 on the sums, bfloat16 out
     GemmParams p {};
     p.K = K;
@@ -1755,8 +1767,8 @@ CHIBI_API int chibi_gemm_bf16_fused(const void* x, const void* w, void* out, int
     p.residual = residual;
     p.res_stride = res_stride;
     p.error = error;
-    p.swiglu = epilogue == 1 ? 1 : 0;
-    p.act = epilogue >= 2 ? epilogue - 1 : 0;
+    p.swiglu = epilogue == 1 ? 1 : (epilogue == 6 ? 2 : 0);
+    p.act = epilogue >= 2 && epilogue <= 5 ? epilogue - 1 : 0;
     p.k_blocks_total = (K + TILE_K - 1) / TILE_K;
     CUtensorMap ma, mb;
     if (M <= 64)
@@ -1785,7 +1797,7 @@ CHIBI_API int chibi_gemm_bf16_fused(const void* x, const void* w, void* out, int
 
 // Many rows with an RMSNorm folded into the products around it (see GemmParams).  `scale`
 // (may be null) describes the factor that x lacks; `norm` (may be null) asks for the norm output of
-// the completed residual.  epilogue 1: SwiGLU as in chibi_gemm_bf16_fused.  Only the kernel for more
+// the completed residual.  epilogue 1, 6: gated products as in chibi_gemm_bf16_fused.  Only the kernel for more
 // than FEW_ROWS_MAX rows with whole tiles of 128 or 256 columns does this: CHIBI_ERR_UNSUPPORTED
 // otherwise, and the caller applies the norm or the factor with kernels of their own.
 struct ChibiRowScale {
@@ -1840,9 +1852,9 @@ CHIBI_API int chibi_gemm_bf16_rows(const void* x, const void* w, void* out, int 
         || (reinterpret_cast<uintptr_t>(out) & 15) || (residual && (reinterpret_cast<uintptr_t>(residual) & 15)))
         return CHIBI_ERR_UNSUPPORTED;
     const int bn = many_rows_tile_width(M, N, K);
-    if (epilogue < 0 || epilogue > 5)
+    if (epilogue < 0 || epilogue > 6)
         return CHIBI_ERR_ARGUMENT;
-    if (epilogue >= 2 && (out_type != CHIBI_BF16 || residual || norm || heads))
+    if (epilogue >= 2 && epilogue <= 5 && (out_type != CHIBI_BF16 || residual || norm || heads))
         return CHIBI_ERR_UNSUPPORTED;      // epilogue 2 .. 5: activation 0 .. 3 on the sums, bfloat16 out
     if (heads) {
         const bool caches = heads->k_cache != nullptr;
@@ -1866,8 +1878,8 @@ CHIBI_API int chibi_gemm_bf16_rows(const void* x, const void* w, void* out, int 
     p.residual = residual;
     p.res_stride = res_stride;
     p.error = error;
-    p.swiglu = epilogue == 1 ? 1 : 0;
-    p.act = epilogue >= 2 ? epilogue - 1 : 0;
+    p.swiglu = epilogue == 1 ? 1 : (epilogue == 6 ? 2 : 0);
+    p.act = epilogue >= 2 && epilogue <= 5 ? epilogue - 1 : 0;
     p.k_blocks_total = (K + TILE_K - 1) / TILE_K;
     p.k_blocks_per_split = p.k_blocks_total;
     p.swap = 0;
@@ -2088,11 +2100,11 @@ reduce_residual_rmsnorm_cluster_kernel(const float* __restrict__ partial, int sp
     }
 }
 
-// act[m, c] = silu(gate) * up with gate = sum of partial[s][m][c] and up = sum of
+// act[m, c] = act(gate) * up (kind: GemmParams::swiglu) with gate = sum of partial[s][m][c] and up = sum of
 // partial[s][m][I + c], in split order.  Two columns per thread.
 template <typename TO>
 __global__ void reduce_swiglu_kernel(const float* __restrict__ partial, int splits, int M, int inter,
-                                     TO* __restrict__ out, int interleaved)
+                                     TO* __restrict__ out, int interleaved, int kind)
 {
     pdl_enter();
     const int half = inter >> 1;
@@ -2121,8 +2133,8 @@ __global__ void reduce_swiglu_kernel(const float* __restrict__ partial, int spli
             g.x += gq[k].x; g.y += gq[k].y; u.x += uq[k].x; u.y += uq[k].y;
         }
     }
-    out[(size_t)m * inter + 2 * c2] = from_f32<TO>((g.x / (1.f + expf(-g.x))) * u.x);
-    out[(size_t)m * inter + 2 * c2 + 1] = from_f32<TO>((g.y / (1.f + expf(-g.y))) * u.y);
+    out[(size_t)m * inter + 2 * c2] = from_f32<TO>(gate_mul_exact(g.x, u.x, kind));
+    out[(size_t)m * inter + 2 * c2 + 1] = from_f32<TO>(gate_mul_exact(g.y, u.y, kind));
 }
 
 } // namespace chibi
@@ -2181,17 +2193,17 @@ CHIBI_API int chibi_reduce_residual_rmsnorm(const float* partial, int splits, in
 }
 
 CHIBI_API int chibi_reduce_swiglu(const float* partial, int splits, int M, int inter, void* out,
-                                  int out_type, int interleaved, cudaStream_t stream)
+                                  int out_type, int interleaved, int kind, cudaStream_t stream)
 {
     if (M <= 0)
         return CHIBI_OK;
     if (inter % 2 != 0 || M > 65535 || splits < 1 || (reinterpret_cast<uintptr_t>(partial) & 7)
-        || (interleaved && inter % 64 != 0))
+        || (interleaved && inter % 64 != 0) || kind < 1 || kind > 2)
         return CHIBI_ERR_UNSUPPORTED;
     const dim3 grid((inter / 2 + 255) / 256, M);
     CHIBI_DISPATCH_TYPE(out_type, TO, {
         launch(reduce_swiglu_kernel<TO>, dim3(grid), dim3(256), 0, stream, partial, splits, M, inter, (TO*)out,
-               interleaved);
+               interleaved, kind);
     });
     return launch_status();
 }

@@ -19,6 +19,7 @@
 #define CHIBI_UNIT hybrid_ops
 #define CHIBI_UNIT_ID 12
 #include "common.cuh"
+#include "row_access.cuh"
 
 namespace chibi {
 
@@ -89,82 +90,129 @@ __global__ void add_weighted_kernel(float* __restrict__ acc, const float* __rest
 }
 
 // ---------------------------------------------------------------- heads: bias, norm, rotation, append
+struct HeadsPrepare {
+    const float* bias;               // over the row, or null
+    const float* q_norm;             // [d], or null
+    const float* k_norm;
+    float eps;                       // q and k heads are normalised if there are weights or unit_norm is set
+    int unit_norm;
+    float temperature;               // q times 1 + temperature * ln(floor((position + 1) / every) + 1); every 0: off
+    int every;
+    const float* inv_freq;
+    int rot;
+    const int* positions;
+    const int* seq_of_token;
+    const int* seq_rows;
+    const int* table;
+    long long table_stride;
+    long long tokens;
+    int nq, nk, nv, d, dv, page_size, num_pages;
+    int* error;
+};
+
 // One warp per (token, job); the jobs of a token are its nq query heads, nk key heads and nv value heads.
 // Shared memory: d floats per warp.
-template <typename TX, typename TC>
+template <typename TX, typename TC, int V>
 __global__ void __launch_bounds__(128)
-heads_prepare_append_kernel(const TX* __restrict__ proj, long long stride, const float* __restrict__ bias,
-                            const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
-                            const float* __restrict__ inv_freq, int rot, const int* __restrict__ positions,
-                            const int* __restrict__ seq_of_token, const int* __restrict__ seq_rows,
-                            const int* __restrict__ table, long long table_stride, TX* __restrict__ q_out,
-                            TC* __restrict__ k_cache, TC* __restrict__ v_cache, long long tokens, int nq, int nk,
-                            int nv, int d, int dv, int page_size, int num_pages, int* __restrict__ error)
+heads_prepare_append_kernel(const HeadsPrepare p, const ProductRows<TX> rows, TC* __restrict__ q_out,
+                            TC* __restrict__ k_cache, TC* __restrict__ v_cache)
 {
     pdl_enter();
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int jobs = nq + (k_cache ? nk + nv : 0);
-    const long long job = (long long)blockIdx.x * (blockDim.x >> 5) + warp;
-    if (job >= tokens * jobs)
+    const unsigned jobs = (unsigned)(p.nq + (k_cache ? p.nk + p.nv : 0));
+    const unsigned job = blockIdx.x * 4u + (unsigned)warp;
+    if (job >= (unsigned)p.tokens * jobs)
         return;
     const long long t = job / jobs;
-    const int j = (int)(job - t * jobs);
-    const int pos = positions[t];
-    const TX* row = proj + (size_t)t * stride;
-    long long slot_row = -1;                                     // (page, position in page) of this token
-    if (j >= nq) {
-        const int seq = seq_of_token[t];
-        const int page = table[(size_t)(seq_rows ? seq_rows[seq] : seq) * table_stride + pos / page_size];
-        if (page < 0 || page >= num_pages) {
-            if (error && lane == 0)
-                atomicExch(error, 3);
+    const int j = (int)(job % jobs);
+    const int d = p.d, dv = p.dv;
+    const bool is_v = j >= p.nq + p.nk;
+    const int col0 = is_v ? (p.nq + p.nk) * d + (j - p.nq - p.nk) * dv : j * d;
+    const int size = is_v ? dv : d;
+    float first[V];                                              // on its way while the page is looked up
+    if (lane * V < size)
+        rows.template load<V>(first, t, col0 + lane * V);
+    const int pos = p.positions[t];
+    long long page = -1;                                         // the page of this token's keys and values
+    if (j >= p.nq) {
+        const int seq = p.seq_of_token[t];
+        page = p.table[(p.seq_rows ? p.seq_rows[seq] : seq) * p.table_stride + pos / p.page_size];
+        if (page < 0 || page >= p.num_pages) {
+            if (p.error && lane == 0)
+                atomicExch(p.error, 3);
             return;
         }
-        slot_row = (long long)page;
     }
-    if (j >= nq + nk) {                                          // a value head: bias and copy
-        const int h = j - nq - nk;
-        const int col0 = nq * d + nk * d + h * dv;
-        TC* dst = v_cache + (((size_t)slot_row * nv + h) * page_size + pos % page_size) * dv;
-        for (int c = lane; c < dv; c += 32)
-            dst[c] = from_f32<TC>(to_f32(row[col0 + c]) + (bias ? bias[col0 + c] : 0.f));
+    if (is_v) {                                                  // a value head: bias and copy
+        const int h = j - p.nq - p.nk;
+        TC* dst = v_cache + ((page * p.nv + h) * p.page_size + pos % p.page_size) * dv;
+        for (int c = lane * V; c < dv; c += 32 * V) {
+            float v[V];
+            if (c >= 32 * V)
+                rows.template load<V>(v, t, col0 + c);
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                if (c < 32 * V)
+                    v[i] = first[i];
+                if (p.bias)
+                    v[i] += p.bias[col0 + c + i];
+            }
+            store_values<TC, V>(dst + c, v);
+        }
         return;
     }
-    const bool is_q = j < nq;
-    const int col0 = is_q ? j * d : nq * d + (j - nq) * d;
+    const bool is_q = j < p.nq;
     float* xs = smem + (size_t)warp * d;
     float ssq = 0.f;
-    for (int c = lane; c < d; c += 32) {
-        const float v = to_f32(row[col0 + c]) + (bias ? bias[col0 + c] : 0.f);
-        xs[c] = v;
-        ssq = fmaf(v, v, ssq);
+    for (int c = lane * V; c < d; c += 32 * V) {
+        float v[V];
+        if (c >= 32 * V)
+            rows.template load<V>(v, t, col0 + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            if (c < 32 * V)
+                v[i] = first[i];
+            if (p.bias)
+                v[i] += p.bias[col0 + c + i];
+            ssq = fmaf(v[i], v[i], ssq);
+        }
+        store_values<float, V>(xs + c, v);
     }
-    const float* w = is_q ? q_norm : k_norm;
-    if (w) {
-        ssq = warp_sum(ssq);
-        const float inv = 1.f / sqrtf(ssq / (float)d + eps);
-        for (int c = lane; c < d; c += 32)
-            xs[c] = xs[c] * inv * w[c];
-    }
+    const float* w = is_q ? p.q_norm : p.k_norm;
+    float inv = 1.f;
+    if (w || p.unit_norm)
+        inv = 1.f / sqrtf(warp_sum(ssq) / (float)d + p.eps);
+    float heat = 1.f;
+    if (is_q && p.every > 0)
+        heat = 1.f + p.temperature * logf((float)((pos + 1) / p.every + 1));
     __syncwarp();
-    const int half = rot >> 1;
+    const int half = p.rot >> 1;
     for (int c = lane; c < half; c += 32) {
         float sn, cs;
-        sincosf((float)pos * inv_freq[c], &sn, &cs);
-        const float u = xs[c], v = xs[c + half];
+        sincosf((float)pos * p.inv_freq[c], &sn, &cs);
+        float u = xs[c] * inv, v = xs[c + half] * inv;
+        if (w)
+            u *= w[c], v *= w[c + half];
         xs[c] = u * cs - v * sn;
         xs[c + half] = v * cs + u * sn;
     }
     __syncwarp();
-    if (is_q) {
-        TX* dst = q_out + ((size_t)t * nq + j) * d;
-        for (int c = lane; c < d; c += 32)
-            dst[c] = from_f32<TX>(xs[c]);
-    } else {
-        TC* dst = k_cache + (((size_t)slot_row * nk + (j - nq)) * page_size + pos % page_size) * d;
-        for (int c = lane; c < d; c += 32)
-            dst[c] = from_f32<TC>(xs[c]);
+    TC* dst = is_q ? q_out + (t * p.nq + j) * d
+                   : k_cache + ((page * p.nk + (j - p.nq)) * p.page_size + pos % p.page_size) * d;
+    for (int c = lane * V; c < d; c += 32 * V) {
+        float v[V];
+        load_values<float, V>(v, xs + c);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            if (c + i >= p.rot) {                                // (the rotated features are finished)
+                v[i] *= inv;
+                if (w)
+                    v[i] *= w[c + i];
+            }
+            v[i] *= heat;
+        }
+        store_values<TC, V>(dst + c, v);
     }
 }
 
@@ -680,34 +728,41 @@ CHIBI_API int chibi_add_weighted(float* acc, const float* a, float wa, const flo
     return launch_status();
 }
 
-CHIBI_API int chibi_heads_prepare_append(const void* proj, int x_type, long long stride, const float* bias,
-                                         const float* q_norm, const float* k_norm, float eps, const float* inv_freq,
-                                         int rot, const int* positions, const int* seq_of_token, const int* seq_rows,
-                                         const int* table, long long table_stride, void* q_out, void* k_cache,
-                                         void* v_cache, int cache_type, long long tokens, int nq, int nk, int nv, int d,
-                                         int dv, int page_size, int num_pages, int* error, cudaStream_t stream)
+// `rows`: [tokens] rows q | k | v of a product; splits > 1: 32-bit partial sums, split_stride apart.  q_out and the
+// caches have type `out_type`.
+CHIBI_API int chibi_heads_prepare_append(const void* rows, int x_type, long long stride, int splits,
+                                         long long split_stride, const float* bias, const float* q_norm,
+                                         const float* k_norm, float eps, int unit_norm, float temperature, int every,
+                                         const float* inv_freq, int rot, const int* positions, const int* seq_of_token,
+                                         const int* seq_rows, const int* table, long long table_stride, void* q_out,
+                                         void* k_cache, void* v_cache, int out_type, long long tokens, int nq, int nk,
+                                         int nv, int d, int dv, int page_size, int num_pages, int* error,
+                                         cudaStream_t stream)
 {
     if (tokens <= 0)
         return CHIBI_OK;
-    if (!proj || !q_out || nq <= 0 || d <= 0 || rot < 0 || rot > d || rot % 2 != 0 || (rot > 0 && !inv_freq)
+    if (!rows || !q_out || nq <= 0 || d <= 0 || rot < 0 || rot > d || rot % 2 != 0 || (rot > 0 && !inv_freq) || every < 0
+        || splits < 1 || (splits > 1 && x_type != CHIBI_F32)
         || (k_cache && (!v_cache || !table || nk <= 0 || nv <= 0 || dv <= 0 || page_size <= 0)))
         return CHIBI_ERR_ARGUMENT;
-    if (d > 4096)
-        return CHIBI_ERR_UNSUPPORTED;
-    const int warps = 4;
     const long long jobs = tokens * (nq + (k_cache ? nk + nv : 0));
-    const long long blocks = (jobs + warps - 1) / warps;
-    if (blocks > 2147483647LL)
+    if (d > 4096 || jobs > 2147483647LL)
         return CHIBI_ERR_UNSUPPORTED;
-    const size_t smem = (size_t)warps * d * sizeof(float);
-    CHIBI_DISPATCH_TYPE(x_type, TX, CHIBI_DISPATCH_TYPE(cache_type, TC, {
+    const HeadsPrepare p { bias, q_norm, k_norm, eps, unit_norm, temperature, every, inv_freq, rot, positions,
+                           seq_of_token, seq_rows, table, table_stride, tokens, nq, nk, nv, d, dv, page_size, num_pages,
+                           error };
+    const size_t smem = (size_t)4 * d * sizeof(float);
+    const uintptr_t unit = out_type == CHIBI_F32 ? 16 : 8;
+    const bool fours = d % 4 == 0 && (!k_cache || dv % 4 == 0) && rows_in_fours(rows, x_type, stride, split_stride)
+                       && reinterpret_cast<uintptr_t>(q_out) % unit == 0 && reinterpret_cast<uintptr_t>(k_cache) % unit == 0
+                       && reinterpret_cast<uintptr_t>(v_cache) % unit == 0;
+    CHIBI_DISPATCH_TYPE(x_type, TX, CHIBI_DISPATCH_TYPE(out_type, TC, {
+        auto kernel = fours ? heads_prepare_append_kernel<TX, TC, 4> : heads_prepare_append_kernel<TX, TC, 1>;
+        const ProductRows<TX> source { (const TX*)rows, stride, splits, split_stride };
         if (smem > 48 * 1024)
-            cudaFuncSetAttribute(heads_prepare_append_kernel<TX, TC>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                 (int)smem);
-        launch(heads_prepare_append_kernel<TX, TC>, dim3((unsigned)blocks), dim3(warps * 32), smem, stream,
-               (const TX*)proj, stride, bias, q_norm, k_norm, eps, inv_freq, rot, positions, seq_of_token, seq_rows,
-               table, table_stride, (TX*)q_out, (TC*)k_cache, (TC*)v_cache, tokens, nq, nk, nv, d, dv, page_size,
-               num_pages, error);
+            cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        launch(kernel, dim3((unsigned)((jobs + 3) / 4)), dim3(128), smem, stream, p, source, (TC*)q_out, (TC*)k_cache,
+               (TC*)v_cache);
     }));
     return launch_status();
 }

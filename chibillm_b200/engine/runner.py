@@ -57,6 +57,8 @@ def make_runtime(dtype, device="cuda:0", kernels=None, spec=None) -> Runtime:
             head_dims = set()
             for layer in spec.layers:
                 for m in mixers(layer.mixer):
+                    if m.kind == "latent_attention":
+                        head_dims.add(m.rope_dim + m.kv_rank)        # one key head whose rows are the values too
                     if m.kind != "attention":
                         continue
                     dv = getattr(m, "value_dim", None) or m.head_dim

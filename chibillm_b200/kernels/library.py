@@ -42,7 +42,7 @@ _SIGNATURES = {
         "chibi_gemm_bf16_fused": [P, P, P, I, P, I, I, I, L, L, L, L, I, P, P],
         "chibi_gemm_bf16_partial": [P, P, I, I, I, L, L, P, L, I, P, P],
         "chibi_reduce_residual_rmsnorm": [P, I, I, I, P, L, P, I, P, I, L, F, F, P],
-        "chibi_reduce_swiglu": [P, I, I, I, P, I, I, P],
+        "chibi_reduce_swiglu": [P, I, I, I, P, I, I, I, P],
         "chibi_qk_norm_rope_append_partial": [P, I, L, L, P, P, P, P, P, I, P, P, P, P, P, I, I, I, I, I,
                                               I, I, F, F, I, P, P],
         "chibi_attention_generic": [P, I, P, P, I, P, P, I, P, P, P, P, P, L, I, I, I, I, I, I, F, I, I, F, P, P, P, P, P],
@@ -83,7 +83,11 @@ _SIGNATURES = {
         "chibi_bigram_embed": [P, P, I, P, P, P, P, P, P, L, I, I, L, L, P],
         "chibi_stream_enter": [P, P, P, L, I, P],
         "chibi_add_weighted": [P, P, F, P, F, L, P],
-        "chibi_heads_prepare_append": [P, I, L, P, P, P, F, P, I, P, P, P, P, L, P, P, P, I, L, I, I, I, I, I, I, I, P, P],
+        "chibi_heads_prepare_append": [P, I, L, I, L, P, P, P, F, I, F, I, P, I, P, P, P, P, L, P, P, P, I, L, I, I, I, I, I,
+                                       I, I, P, P],
+        "chibi_position_rows": [P, F, P, I, I, P, P, F, L, I, P, P],
+        "chibi_latent_heads_append": [P, I, L, I, L, P, P, I, P, F, P, I, I, I, P, P, P, P, P, L, I, I, L, P, P],
+        "chibi_head_gate": [P, I, P, L, I, I, P],
         "chibi_differential_combine": [P, P, I, L, F, F, F, P, L, I, I, I, P],
         "chibi_state_space_scan": [P, I, L, P, L, P, P, P, P, P, P, P, I, I, I, I, I, P],
         "chibi_gated_group_rms": [P, P, I, L, P, F, P, L, I, I, P],

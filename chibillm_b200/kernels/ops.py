@@ -88,9 +88,11 @@ class ScaledRows:
     x * (w + offset) in bfloat16 and ``ssq`` [rows, parts] sums of squares of x, so
     that RMSNorm(x)[m] = tensor[m] * rsqrt(sum(ssq[m]) / n + eps).  The factor
     commutes with a matrix product, and ``linear`` / ``linear_swiglu`` apply it to
-    their sums; ``materialise`` applies it in place for any other reader."""
+    their sums; ``materialise`` applies it in place (once) for any other reader, and for
+    every reader after that."""
 
     def __init__(self, kernels, tensor: torch.Tensor, ssq: torch.Tensor, parts: int, eps: float, n: int):
+        self.applied = False             # the factor is in ``tensor`` already
         self.kernels, self.tensor, self.ssq, self.parts, self.eps, self.n = kernels, tensor, ssq, parts, eps, n
 
     @property
@@ -102,7 +104,9 @@ class ScaledRows:
         return self.tensor.dtype
 
     def materialise(self) -> torch.Tensor:
-        self.kernels.scale_rows(self)
+        if not self.applied:
+            self.kernels.scale_rows(self)
+            self.applied = True
         return self.tensor
 
 
@@ -293,14 +297,16 @@ class CudaKernels:
             self.scratch_generation += 1
         return buf
 
-    def _linear_of_scaled(self, x: ScaledRows, w: torch.Tensor, out: torch.Tensor, swiglu: bool,
+    def _linear_of_scaled(self, x: ScaledRows, w: torch.Tensor, out: torch.Tensor, swiglu,
                           activation: Optional[str] = None) -> bool:
-        """out = (the factor of each row) * (x.tensor @ w^T), with SwiGLU or an
-        activation if asked, from the kernel for many rows; False if it does not take
+        """out = (the factor of each row) * (x.tensor @ w^T), with a gate (``swiglu``: an epilogue
+        of _GATED_EPILOGUES or False) or an activation if asked, from the kernel for many rows; False if it does not take
         the shapes."""
         t = x.tensor
         M, K = t.shape
         N = w.shape[0]
+        if x.applied:
+            return False
         if not (self.use_tensor_cores and M > self.few_rows_max and N % 128 == 0 and w.dtype == torch.bfloat16
                 and out.dtype == torch.bfloat16 and w.shape[1] == K
                 and out.shape == (M, N // 2 if swiglu else N)):
@@ -311,7 +317,7 @@ class CudaKernels:
         scale = library.RowScale(_ptr(x.ssq), x.parts, float(x.eps), x.n)
         status = self.lib.chibi_gemm_bf16_rows(
             _ptr(t), _ptr(w), _ptr(out), BF16, None, M, N, K, t.stride(0), w.stride(0), out.stride(0), 0,
-            1 if swiglu else (2 + self._EPILOGUE_ACTIVATIONS[activation] if activation is not None else 0),
+            int(swiglu) if swiglu else (2 + self._EPILOGUE_ACTIVATIONS[activation] if activation is not None else 0),
             ctypes.byref(scale), None, None, _ptr(self.error), self._stream())
         if status == -2:
             return False
@@ -442,7 +448,7 @@ class CudaKernels:
             self.lib.chibi_gemm_reset_stream_counters(self._stream())
             what = {1: "a token id outside the vocabulary", 2: "a page id outside the pool (append)",
                     3: "a page id outside the pool (attention)",
-                    4: "a block-table update outside the table",
+                    4: "a block-table update outside the table", 6: "a position outside the table of position rows",
                     5: "a table entry outside its range (an expert, or a token id of a per-layer token input)",
                     11: "a wait that ran out (matrix product: loader)",
                     12: "a wait that ran out (matrix product: tensor-core issuer)",
@@ -531,6 +537,40 @@ class CudaKernels:
         return PendingSum(self, buf[:splits * M * N].view(splits, M, N), splits, M, N,
                           self._partial_turn, self._partial_stamps[self._partial_turn])
 
+    def linear_pair(self, x1: torch.Tensor, w1: torch.Tensor, x2: torch.Tensor, w2: torch.Tensor,
+                    residual: torch.Tensor):
+        """residual += x1 @ w1^T + x2 @ w2^T, the last of it left pending (an object with ``add_into``).  Two
+        products of few rows whose K ranges are split leave their partial sums side by side in one
+        array, so that whoever adds them up does it in one go."""
+        M, N = residual.shape
+        if self.use_tensor_cores and self.fuse_split_products and N % 4 == 0 \
+                and all(t.dtype == torch.bfloat16 for t in (x1, w1, x2, w2)) and tuple(x1.shape) == (M, w1.shape[1]) \
+                and tuple(x2.shape) == (M, w2.shape[1]) and w1.shape[0] == N and w2.shape[0] == N:
+            splits = [self.lib.chibi_gemm_bf16_splits_capped(M, N, w.shape[1], 0) for w in (w1, w2)]
+            if min(splits) > 1:
+                for t in (x1, w1, x2, w2):
+                    _need_cuda(t)
+                    _rows_contiguous(t, "linear_pair")
+                buf = self._partial_buffer(sum(splits) * M * N)
+                at, taken = 0, True
+                for x, w, s in ((x1, w1, splits[0]), (x2, w2, splits[1])):
+                    part = buf[at * M * N:(at + s) * M * N]
+                    status = self.lib.chibi_gemm_bf16_partial(_ptr(x), _ptr(w), M, N, w.shape[1], x.stride(0), w.stride(0),
+                                                              _ptr(part), part.numel(), 0, _ptr(self.error),
+                                                              self._stream())
+                    if status == -2:
+                        taken = False
+                        break
+                    _check(status, "linear_pair")
+                    self.launches += 1
+                    self.tensor_core_calls += 1
+                    at += s
+                if taken:
+                    return PendingSum(self, buf[:at * M * N].view(at, M, N), at, M, N, self._partial_turn,
+                                      self._partial_stamps[self._partial_turn])
+        self.linear(x1, w1, residual, residual=residual)
+        return self.linear(x2, w2, residual, residual=residual, defer=True)
+
     @staticmethod
     def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> Optional[torch.Tensor]:
         """[gate; up] rearranged for ``linear_swiglu``: blocks of 64 gate rows, each
@@ -542,12 +582,16 @@ class CudaKernels:
             return None
         return torch.stack([gate.view(inter // 64, 64, k), up.view(inter // 64, 64, k)], dim=1).reshape(2 * inter, k).contiguous()
 
-    def linear_swiglu(self, x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor) -> bool:
-        """out[M, I] = silu(x @ gate^T) * (x @ up^T) in one kernel, with the weights
+    # gated products: the gate's activation -> (epilogue of the kernel for many rows, kind of the reduction)
+    _GATED_EPILOGUES = {"silu": (1, 1), "gelu_tanh": (6, 2)}
+
+    def linear_swiglu(self, x: torch.Tensor, w_interleaved: torch.Tensor, out: torch.Tensor, kind: str = "silu") -> bool:
+        """out[M, I] = act(x @ gate^T) * (x @ up^T) in one kernel (``kind``: "silu" or "gelu_tanh"), with the weights
         as ``interleave_gate_up`` arranges them.  False if the kernel refuses the
         shapes (the caller then takes the two-kernel way)."""
+        epilogue = self._GATED_EPILOGUES[kind][0]
         if isinstance(x, ScaledRows):
-            if self._linear_of_scaled(x, w_interleaved, out, swiglu=True):
+            if self._linear_of_scaled(x, w_interleaved, out, swiglu=epilogue):
                 return True
             x = x.materialise()
         _need_cuda(x, w_interleaved, out)
@@ -570,11 +614,11 @@ class CudaKernels:
                 self.linear(x, w_interleaved, buf[:M * N].view(M, N))
                 pending = PendingSum(self, buf[:M * N].view(1, M, N), 1, M, N, self._partial_turn,
                                      self._partial_stamps[self._partial_turn])
-            self.reduce_swiglu(pending, out, interleaved=True)
+            self.reduce_swiglu(pending, out, interleaved=True, kind=kind)
             return True
         status = self.lib.chibi_gemm_bf16_fused(
             _ptr(x), _ptr(w_interleaved), _ptr(out), BF16, None, M, N, K, x.stride(0),
-            w_interleaved.stride(0), out.stride(0), 0, 1, _ptr(self.error), self._stream())
+            w_interleaved.stride(0), out.stride(0), 0, epilogue, _ptr(self.error), self._stream())
         if status == -2:
             return False
         _check(status, "linear_swiglu")
@@ -614,8 +658,9 @@ class CudaKernels:
         self.launches += 1
         _check(status, "reduce_residual_rmsnorm")
 
-    def reduce_swiglu(self, pending: PendingSum, out: torch.Tensor, interleaved: bool = False) -> None:
-        """out = silu(gate) * up from the pending [gate | up] product (or, with
+    def reduce_swiglu(self, pending: PendingSum, out: torch.Tensor, interleaved: bool = False,
+                      kind: str = "silu") -> None:
+        """out = act(gate) * up from the pending [gate | up] product (or, with
         ``interleaved``, from a product with ``interleave_gate_up`` weights)."""
         _need_cuda(out)
         inter = pending.N // 2
@@ -624,7 +669,7 @@ class CudaKernels:
         self.launches += 1
         _check(self.lib.chibi_reduce_swiglu(_ptr(pending.partial), pending.splits, pending.M, inter,
                                             _ptr(out), _code(out), 1 if interleaved else 0,
-                                            self._stream()), "reduce_swiglu")
+                                            self._GATED_EPILOGUES[kind][1], self._stream()), "reduce_swiglu")
 
     def qk_norm_rope_append_partial(self, pending: PendingSum, q_out, k_cache, v_cache, q_norm_w, k_norm_w,
                                     inv_freq, rotary_dim, eps, norm_offset, positions, seq_of_token,
@@ -1746,21 +1791,30 @@ class CudaKernels:
                              inv_freq: Optional[torch.Tensor], rotary_dim: int, positions: torch.Tensor,
                              seq_of_token: torch.Tensor, block_table: Optional[torch.Tensor], nq: int, nk: int,
                              nv: int, d: int, dv: int, page_size: int,
-                             seq_rows: Optional[torch.Tensor] = None) -> None:
-        """Per head of a row q | k | v ([T, >= nq d + nk d + nv dv]; [T, >= nq d] without a cache):
-        + bias (float32 over the row, or None); q and k heads divided by their root mean square and
-        multiplied by ``q_norm`` / ``k_norm`` (float32 [d], both or none); the first ``rotary_dim``
-        features rotated; q -> q_out, k -> [pages, nk, page, d], v -> [pages, nv, page, dv]."""
-        _need_cuda(proj, q_out, k_cache, v_cache, bias, q_norm, k_norm, inv_freq, positions, seq_of_token,
-                   block_table, seq_rows)
-        _rows_contiguous(proj, "heads_prepare_append: proj")
-        T = proj.shape[0]
+                             seq_rows: Optional[torch.Tensor] = None, unit_norm_eps: Optional[float] = None,
+                             temperature=None) -> None:
+        """Per head of a row q | k | v ([T, >= nq d + nk d + nv dv], an array or a PendingSum; [T, >= nq d] without a
+        cache): + bias (float32 over the row, or None); q and k heads divided by their root mean square and
+        multiplied by ``q_norm`` / ``k_norm`` (float32 [d], both or none; ``unit_norm_eps``: divided without
+        weights); the first ``rotary_dim`` features rotated; q times 1 + c ln(floor((position + 1) / every) + 1)
+        with ``temperature`` = (c, every); q -> q_out, k -> [pages, nk, page, d], v -> [pages, nv, page, dv]."""
+        rows, code, stride, splits, split_stride, T, columns = self._product_rows(proj, q_out, "heads_prepare_append")
+        _need_cuda(q_out, k_cache, v_cache, bias, q_norm, k_norm, inv_freq, positions, seq_of_token, block_table,
+                   seq_rows)
         append = k_cache is not None
         width = nq * d + ((nk * d + nv * dv) if append else 0)
-        if proj.shape[1] < width or not q_out.is_contiguous() or q_out.shape != (T, nq * d) or q_out.dtype != proj.dtype:
+        if columns < width or not q_out.is_contiguous() or q_out.shape != (T, nq * d) \
+                or (append and k_cache.dtype != q_out.dtype):
             raise KernelError("heads_prepare_append: proj / q_out shapes or types")
         if (q_norm is None) != (k_norm is None):
             raise KernelError("heads_prepare_append: give both norm weights or none")
+        if unit_norm_eps is not None:
+            if q_norm is not None:
+                raise KernelError("heads_prepare_append: a norm with or without weights, not both")
+            eps = unit_norm_eps
+        coef, every = temperature if temperature is not None else (0.0, 0)
+        if temperature is not None and int(every) < 1:
+            raise KernelError("heads_prepare_append: the temperature's step is a positive number of positions")
         for t, size, what in ((bias, width, "bias"), (q_norm, d, "q_norm"), (k_norm, d, "k_norm")):
             if t is not None and (t.dtype != torch.float32 or t.numel() < size or not t.is_contiguous()):
                 raise KernelError(f"heads_prepare_append: {what} must be contiguous float32 of {size} values")
@@ -1777,11 +1831,86 @@ class CudaKernels:
             table_stride = block_table.stride(0)
         self.launches += 1
         _check(self.lib.chibi_heads_prepare_append(
-            _ptr(proj), _code(proj), proj.stride(0), _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(eps),
-            _ptr(inv_freq) if rotary_dim else None, int(rotary_dim), _ptr(positions), _ptr(seq_of_token),
+            rows, code, stride, splits, split_stride, _ptr(bias), _ptr(q_norm), _ptr(k_norm), float(eps),
+            1 if unit_norm_eps is not None else 0, float(coef), int(every), _ptr(inv_freq) if rotary_dim else None, int(rotary_dim), _ptr(positions), _ptr(seq_of_token),
             _ptr(seq_rows), _ptr(block_table), table_stride, _ptr(q_out), _ptr(k_cache), _ptr(v_cache),
-            _code(k_cache) if append else F32, T, nq, nk, nv, d, dv, page_size, num_pages, _ptr(self.error),
-            self._stream()), "heads_prepare_append")
+            _code(q_out), T, nq, nk, nv, d, dv, page_size, num_pages, _ptr(self.error), self._stream()),
+            "heads_prepare_append")
+
+    @staticmethod
+    def _product_rows(proj, out: torch.Tensor, what: str):
+        """A product's rows as a kernel that finishes them reads them, an array or partial sums (then
+        32-bit, for bfloat16 outputs): pointer, type, row stride, splits, split stride, rows, columns."""
+        if isinstance(proj, PendingSum):
+            if out.dtype != torch.bfloat16:
+                raise KernelError(f"{what}: partial sums belong to bfloat16 outputs")
+            return _ptr(proj.partial), F32, proj.N, proj.splits, proj.M * proj.N, proj.M, proj.N
+        _need_cuda(proj)
+        _rows_contiguous(proj, f"{what}: proj")
+        if proj.dtype != out.dtype:
+            raise KernelError(f"{what}: the rows have the outputs' type")
+        return _ptr(proj), _code(proj), proj.stride(0), 1, 0, proj.shape[0], proj.shape[1]
+
+    def latent_heads_append(self, proj, q_out: torch.Tensor, k_cache: Optional[torch.Tensor],
+                            kv_norm: Optional[torch.Tensor], eps: float, inv_freq: torch.Tensor, heads: int,
+                            kv_rank: int, rot: int, gates: Optional[torch.Tensor], positions: torch.Tensor,
+                            seq_of_token: torch.Tensor, block_table: Optional[torch.Tensor], page_size: int,
+                            seq_rows: Optional[torch.Tensor] = None) -> None:
+        """From rows q | c | k_rot | g (an array or a PendingSum; q: ``heads`` times rot + kv_rank columns; c | k_rot
+        only with a cache; g only with ``gates``): q_out takes q with every head's first ``rot`` features
+        rotated; the cache row of the token's position ([pages, 1, page, rot + kv_rank]) the rotated
+        k_rot, then RMSNorm(c) * kv_norm; ``gates`` [T, heads] float32 the sigmoid of g."""
+        rows, code, stride, splits, split_stride, T, columns = self._product_rows(proj, q_out, "latent_heads_append")
+        _need_cuda(q_out, k_cache, kv_norm, inv_freq, gates, positions, seq_of_token, block_table, seq_rows)
+        append = k_cache is not None
+        kd = rot + kv_rank
+        width = heads * kd + (kd if append else 0) + (heads if gates is not None else 0)
+        if columns < width or q_out.shape != (T, heads * kd) or not q_out.is_contiguous():
+            raise KernelError("latent_heads_append: proj / q_out shapes")
+        if inv_freq.dtype != torch.float32 or inv_freq.numel() < rot // 2:
+            raise KernelError("latent_heads_append: inv_freq must hold rot/2 float32 values")
+        if gates is not None and (gates.dtype != torch.float32 or gates.shape != (T, heads) or not gates.is_contiguous()):
+            raise KernelError("latent_heads_append: the gates are contiguous float32 [T, heads]")
+        num_pages = table_stride = 0
+        if append:
+            if (tuple(k_cache.shape[1:]) != (1, page_size, kd) or not k_cache.is_contiguous() or k_cache.dtype != q_out.dtype
+                    or kv_norm is None or kv_norm.dtype != torch.float32 or kv_norm.numel() != kv_rank):
+                raise KernelError("latent_heads_append: cache or norm weight")
+            num_pages = k_cache.shape[0]
+            _rows_contiguous(block_table, "latent_heads_append: block_table")
+            table_stride = block_table.stride(0)
+        self.launches += 1
+        _check(self.lib.chibi_latent_heads_append(
+            rows, code, stride, splits, split_stride, _ptr(q_out), _ptr(k_cache), _code(q_out), _ptr(kv_norm), float(eps),
+            _ptr(inv_freq), heads, kv_rank, rot, _ptr(gates), _ptr(positions), _ptr(seq_of_token), _ptr(seq_rows),
+            _ptr(block_table), table_stride, page_size, num_pages, T, _ptr(self.error), self._stream()),
+            "latent_heads_append")
+
+    def head_gate(self, x: torch.Tensor, gates: torch.Tensor, heads: int) -> None:
+        """x[t, h, :] *= gates[t, h], in place; x contiguous [T, heads * size], gates float32 [T, heads]."""
+        _need_cuda(x, gates)
+        T = x.shape[0]
+        if not x.is_contiguous() or x.shape[1] % heads or gates.dtype != torch.float32 or gates.shape != (T, heads) \
+                or not gates.is_contiguous():
+            raise KernelError("head_gate: shapes or types")
+        self.launches += 1
+        _check(self.lib.chibi_head_gate(_ptr(x), _code(x), _ptr(gates), T, heads, x.shape[1] // heads, self._stream()),
+               "head_gate")
+
+    def position_rows(self, x: torch.Tensor, factor: float, table: torch.Tensor, positions: torch.Tensor,
+                      weight: Optional[torch.Tensor], eps: float) -> None:
+        """x[t] = factor * x[t] + table[positions[t]]; with a weight (float32 [n]) then divided by its root mean
+        square and multiplied by it.  x contiguous float32 [T, n], in place."""
+        _need_cuda(x, table, positions, weight)
+        T, n = x.shape
+        if x.dtype != torch.float32 or not x.is_contiguous() or table.dim() != 2 or table.shape[1] != n \
+                or not table.is_contiguous() or positions.dtype != torch.int32 or positions.numel() != T \
+                or (weight is not None and (weight.dtype != torch.float32 or weight.shape != (n,) or not weight.is_contiguous())):
+            raise KernelError("position_rows: shapes or types")
+        self.launches += 1
+        _check(self.lib.chibi_position_rows(_ptr(x), float(factor), _ptr(table), _code(table), table.shape[0],
+                                            _ptr(positions), _ptr(weight), float(eps), T, n, _ptr(self.error),
+                                            self._stream()), "position_rows")
 
     def differential_combine(self, att: torch.Tensor, gate: Optional[torch.Tensor], lam: float, eps: float,
                              out_scale: float, out: torch.Tensor, heads: int, dv: int, group: int) -> None:

@@ -22,6 +22,12 @@ table's last row (number ``buckets``) for a sequence's first token (tensor role
 "table"; ``params``: "hidden_size", "buckets", "mul_prev", "mul_cur").  The token
 before a step's first is part of the request's state: the adapter declares a cache
 need of one integer per request.
+
+"position_rows": an input adapter for learned absolute positions: x becomes factor * x plus
+the row of a table (tensor role "table" [``positions``, ``hidden_size``]) at the token's
+position, and, with a tensor role "norm", that sum divided by its root mean square (``eps``
+inside the root) and multiplied by the norm's weight; one kernel (``params``: "hidden_size",
+"positions", "factor", "eps").
 """
 from __future__ import annotations
 
@@ -147,6 +153,35 @@ class Bigram(Adapter):
                                           self.mul_cur)
 
 
+class PositionRows(Adapter):
+    def __init__(self, spec, runtime: Runtime):
+        self.names = spec.names()
+        c = spec.constants()
+        self.hidden, self.positions = int(c["hidden_size"]), int(c["positions"])
+        self.factor, self.eps = float(c.get("factor", 1.0)), float(c.get("eps", 0.0))
+        self.runtime = runtime
+        self.table: torch.Tensor = None
+        self.norm: torch.Tensor = None
+
+    def expected_tensors(self) -> List[TensorSpec]:
+        out = [TensorSpec(self.names["table"], (self.positions, self.hidden), init=("normal", 0.0, 0.02))]
+        if "norm" in self.names:
+            out.append(TensorSpec(self.names["norm"], (self.hidden,)))
+        return out
+
+    def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.table = tensors[self.names["table"]].contiguous()
+        if "norm" in self.names:
+            self.norm = tensors[self.names["norm"]].float().contiguous()
+
+    def launch_key(self, ctx):
+        return ()
+
+    def forward(self, x: torch.Tensor, ctx, turn: int = 0) -> None:
+        self.runtime.kernels.position_rows(x, self.factor, self.table, ctx.positions, self.norm, self.eps)
+
+
+register_adapter("position_rows", PositionRows, replace=True)
 register_adapter("reentry_add", ReentryAdd, replace=True)
 register_adapter("bigram", Bigram, replace=True)
 register_adapter("scale", Scale, replace=True)

@@ -27,7 +27,8 @@ amplitude.  The last two, and a value size of its own, take the plain order of
 kernels: the q | k | v product, one kernel that rotates, normalises and appends,
 attention, the output product.
 
-A sink (``sink``: one learned number per query head in the softmax's denominator)
+A sink (``sink``: one learned number per query head in the softmax's denominator;
+``sink_value``: the same given number for all heads)
 goes to the attention kernels as it is.  Biases on q, k and v, a norm of q and k
 over their whole projections (all heads at once) and a sigmoid gate on the
 concatenated heads (``biases``, ``whole_norm_eps``, ``output_gate``) take an order
@@ -39,7 +40,8 @@ Several score maps per head (``query_maps``; two maps joined as a1 - lambda a2:
 ``differential``), a gate per head (``head_gate``), a bias linear in the distance and
 biases together with a per-head norm take one more order: one product gives
 q | k | v (| the heads' gates); one kernel adds the biases, normalises every q and k
-head with the shared weight, rotates, writes q and appends k and v (the maps of a key
+head (with the shared weight or without one), rotates, multiplies q by a temperature that
+grows with the position (``query_temperature``), writes q and appends k and v (the maps of a key
 head are key heads of the cache that share one value head); attention follows, 32-bit
 where maps are to be subtracted; one kernel joins the maps, normalises and gates; then
 the output product.
@@ -53,7 +55,7 @@ from typing import Dict, List
 
 import torch
 
-from .base import (Mixer, PagedKVNeed, Runtime, TensorSpec, make_position, register_mixer)
+from .base import (HeldProduct, Mixer, PagedKVNeed, Runtime, TensorSpec, make_position, register_mixer)
 
 
 class PagedAttention(Mixer):
@@ -75,13 +77,15 @@ class PagedAttention(Mixer):
         self.maps = int(getattr(spec, "query_maps", 1))
         # the order of the module's last paragraph
         self.prepared = (self.maps > 1 or getattr(spec, "head_gate", False) or spec.distance_bias == "linear"
-                         or (spec.biases and spec.qk_norm is not None))
+                         or (spec.biases and spec.qk_norm is not None) or spec.query_temperature is not None)
         if self.prepared:
-            if spec.tied_values or spec.unit_norm_eps is not None or spec.whole_norm_eps is not None \
+            if spec.tied_values or spec.whole_norm_eps is not None \
                     or spec.output_gate or spec.softcap is not None or not spec.own_kv:
-                raise ValueError("score maps, a gate per head, a linear distance bias and biases with a per-head "
-                                 "norm are not combined with tied values, a norm after the rotation or over the "
+                raise ValueError("score maps, a gate per head, a linear distance bias, a query temperature and biases "
+                                 "with a per-head norm are not combined with tied values, a norm over the "
                                  "whole projection, a gate per feature, a soft cap or a borrowed cache")
+            if spec.unit_norm_eps is not None and spec.biases:
+                raise ValueError("biases are not combined with a norm without a weight")
             if getattr(spec, "differential", None) is not None and self.maps != 2:
                 raise ValueError("differential attention has two score maps per head")
             if self.maps > 1 and getattr(spec, "differential", None) is None:
@@ -98,6 +102,9 @@ class PagedAttention(Mixer):
             raise ValueError("values tied to the keys have the keys' size")
         if spec.tied_values and self.position.feature_order() is not None:
             raise ValueError("values tied to the keys are not combined with a rotation of neighbouring features")
+        if spec.sink and spec.sink_value is not None:
+            raise ValueError("a sink is either learned (sink) or one number (sink_value)")
+        self.has_sink = spec.sink or spec.sink_value is not None
         if spec.unit_norm_eps is not None and spec.qk_norm is not None:
             raise ValueError("a norm of q and k comes either before the rotation (qk_norm) or after it (unit_norm_eps)")
         if self.prepared:
@@ -198,6 +205,9 @@ class PagedAttention(Mixer):
             G, R, d = s.num_kv_heads, s.num_heads // s.num_kv_heads, s.head_dim
             mats[0] = mats[0].view(G, R, M, d, -1).permute(0, 2, 1, 3, 4).reshape(mats[0].shape)
         self.qkv = torch.cat([m.to(mats[0].dtype) for m in mats], dim=0).contiguous()
+        if self.spec.sink_value is not None:
+            self.sink = torch.full((self.spec.num_heads,), float(self.spec.sink_value), dtype=torch.float32,
+                                   device=self.qkv.device)
         if self.spec.sink:
             self.sink = tensors[self.names["sink"]].float().contiguous()
         if self.spec.biases:
@@ -219,6 +229,7 @@ class PagedAttention(Mixer):
     # ---- cache
     accepts_scaled_rows = True       # x goes to the q | k | v product and nowhere else
     can_overwrite = True
+    can_hold = True
 
     def cache_need(self):
         s = self.spec
@@ -231,9 +242,9 @@ class PagedAttention(Mixer):
     def launch_key(self, ctx):
         if self.position.fused_rotation() is None:
             return None                      # an encoding of its own: nothing is promised
-        if self.prepared:
-            return ()                        # the plain attention kernel: nothing is decided on the host
         k = self.runtime.kernels
+        if self.prepared and (self.maps > 1 or self.value_dim != self.spec.head_dim):
+            return ()                        # the plain attention kernel: nothing is decided on the host
         splits = getattr(k, "decode_attention_splits", None)
         if splits is None:
             return None
@@ -241,7 +252,7 @@ class PagedAttention(Mixer):
         return (splits(ctx.num_seqs, s.num_heads, s.num_kv_heads, ctx.max_ctx_len),)
 
     # ---- run
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, cache, overwrite: bool = False):
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, cache, overwrite: bool = False, hold: bool = False):
         s, rt = self.spec, self.runtime
         k = rt.kernels
         T = x.shape[0]
@@ -251,16 +262,16 @@ class PagedAttention(Mixer):
         if writes and not s.own_kv:
             raise ValueError("a layer without key and value projections must read another run step's cache")
         if self.prepared:
-            return self._prepared_attend(x, residual, ctx, cache, overwrite)
+            return self._prepared_attend(x, residual, ctx, cache, overwrite, hold)
         if self.bias_norm_gate:
-            return self._bias_norm_gate_attend(x, residual, ctx, cache, overwrite)
+            return self._bias_norm_gate_attend(x, residual, ctx, cache, overwrite, hold)
         if self.rotate_then_norm:
-            return self._rotate_norm_attend(x, residual, ctx, cache, overwrite)
+            return self._rotate_norm_attend(x, residual, ctx, cache, overwrite, hold)
         width = qw + self.kv_arrays * kw if writes else qw
-        modified = s.softcap is not None or s.distance_bias is not None or s.chunk is not None or s.sink
+        modified = s.softcap is not None or s.distance_bias is not None or s.chunk is not None or self.has_sink
         fused = self.position.fused_rotation()
         if fused is not None and fused[0] is not None and self._heads_from_the_product(x, ctx, cache, fused):
-            return self._attend(residual, ctx, cache, overwrite=overwrite)
+            return self._attend(residual, ctx, cache, overwrite=overwrite, hold=hold)
         split = getattr(k, "linear_partial", None)
         pending = None
         if split is not None and fused is not None and d % 4 == 0:
@@ -285,7 +296,7 @@ class PagedAttention(Mixer):
                             cache.page_size, s.scale, s.window, ctx.max_ctx_len, q_norm_w, k_norm_w, fused[0],
                             fused[1], norm.eps if norm is not None else 0.0,
                             norm.weight_offset if norm is not None else 0.0, writes, ctx.seq_rows):
-                return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
+                return self._output(att, residual, overwrite, hold)
         if fused is None:
             # An encoding the kernels do not know: normalise head by head in
             # place, let the encoding transform q and k, then only copy and append.
@@ -306,9 +317,9 @@ class PagedAttention(Mixer):
             norm.weight_offset if norm is not None else 0.0,
             ctx.positions, ctx.seq_of_token, table if writes else None, nq, nkv, d, cache.page_size,
             ctx.seq_rows)
-        return self._attend(residual, ctx, cache, overwrite=overwrite)
+        return self._attend(residual, ctx, cache, overwrite=overwrite, hold=hold)
 
-    def _rotate_norm_attend(self, x, residual, ctx, cache, overwrite=False):
+    def _rotate_norm_attend(self, x, residual, ctx, cache, overwrite=False, hold=False):
         """The plain order: q | k | v product; per head rotation (with the encoding's
         amplitude), then the norm without a weight; append; attention; output product."""
         s, rt = self.spec, self.runtime
@@ -329,9 +340,9 @@ class PagedAttention(Mixer):
                               s.unit_norm_eps is not None, s.unit_norm_eps or 0.0, ctx.positions, ctx.seq_of_token,
                               ctx.tables[cache.group] if writes else None, nq, nkv, d, dv, cache.page_size,
                               ctx.seq_rows)
-        return self._attend(residual, ctx, cache, overwrite=overwrite)
+        return self._attend(residual, ctx, cache, overwrite=overwrite, hold=hold)
 
-    def _prepared_attend(self, x, residual, ctx, cache, overwrite=False):
+    def _prepared_attend(self, x, residual, ctx, cache, overwrite=False, hold=False):
         """q | k | v (| gates) from one product; biases, per-head norm, rotation and append in one
         kernel; attention with the maps of a head as heads of their own that share the head's
         values; the maps joined, normalised and gated; the output product."""
@@ -343,22 +354,31 @@ class PagedAttention(Mixer):
         inv_freq, rotary_dim = self.position.fused_rotation() or (None, 0)
         if inv_freq is None and s.position.kind != "none":
             raise ValueError("this order of kernels needs a rotation that the kernels apply")
-        proj = ctx.workspace.get("attn.qkv", (T, self.qkv.shape[0]), rt.dtype)
-        k.linear(x, self.qkv, proj)
+        gated = self.gate_columns > 0
+        # few rows: the product's partial sums, for the kernel that finishes the heads (a gate is read later)
+        proj = k.linear_partial(x, self.qkv) if not gated else None
+        if proj is None:
+            proj = ctx.workspace.get("attn.qkv", (T, self.qkv.shape[0]), rt.dtype)
+            k.linear(x, self.qkv, proj)
         q = ctx.workspace.get("attn.q", (T, nq * d), rt.dtype)
         norm = s.qk_norm
+        how = {}
+        if s.unit_norm_eps is not None:
+            how["unit_norm_eps"] = float(s.unit_norm_eps)
+        if s.query_temperature is not None:
+            how["temperature"] = s.query_temperature
         table = ctx.tables[cache.group]
         k.heads_prepare_append(proj, q, cache.keys, cache.values, self.bias,
                                self.q_norm if norm is not None else None, self.k_norm if norm is not None else None,
                                norm.eps if norm is not None else 0.0, inv_freq,
                                rotary_dim if inv_freq is not None else 0, ctx.positions, ctx.seq_of_token, table,
-                               nq, nk, nv, d, dv, cache.page_size, ctx.seq_rows)
+                               nq, nk, nv, d, dv, cache.page_size, ctx.seq_rows, **how)
         extra = {}
         if s.chunk is not None:
             extra["chunk"] = s.chunk
         if dv != d:
             extra["value_dim"] = dv
-        if s.sink:
+        if self.has_sink:
             extra["sink"] = self.sink
         if s.distance_bias == "linear":
             extra["distance_bias"] = (self.slopes, None)
@@ -372,13 +392,13 @@ class PagedAttention(Mixer):
                     ctx.min_q_len, ctx.seq_rows, **extra)
         if joined:
             out = ctx.workspace.get("attn.out", (T, s.num_heads * dv), rt.dtype)
-            gate = proj[:, proj.shape[1] - self.gate_columns:] if self.gate_columns else None
+            gate = proj[:, proj.shape[1] - self.gate_columns:] if gated else None
             k.differential_combine(att, gate, self.lam, s.differential_eps, 1.0 - float(s.differential), out,
                                    s.num_heads, dv, s.num_heads // s.num_kv_heads)
             att = out
-        return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
+        return self._output(att, residual, overwrite, hold)
 
-    def _bias_norm_gate_attend(self, x, residual, ctx, cache, overwrite=False):
+    def _bias_norm_gate_attend(self, x, residual, ctx, cache, overwrite=False, hold=False):
         """q | k | v | gate from one product; biases, the norm over the whole q and k,
         a rotation if the encoding has one, and the append in one kernel; attention;
         the heads times sigmoid(gate); the output product."""
@@ -399,9 +419,9 @@ class PagedAttention(Mixer):
                                ctx.tables[cache.group] if writes else None, nq, nkv, d, dv, cache.page_size,
                                ctx.seq_rows)
         gate = proj[:, proj.shape[1] - self.gate_columns:] if self.gate_columns else None
-        return self._attend(residual, ctx, cache, gate, overwrite=overwrite)
+        return self._attend(residual, ctx, cache, gate, overwrite=overwrite, hold=hold)
 
-    def _attend(self, residual, ctx, cache, gate=None, overwrite=False):
+    def _attend(self, residual, ctx, cache, gate=None, overwrite=False, hold=False):
         """Attention over the cache from the step's q, then the output product, left
         for the next norm to add into the residual."""
         s, rt = self.spec, self.runtime
@@ -418,14 +438,21 @@ class PagedAttention(Mixer):
             extra["chunk"] = s.chunk
         if self.value_dim != d:
             extra["value_dim"] = self.value_dim
-        if s.sink:
+        if self.has_sink:
             extra["sink"] = self.sink
         k.attention(q, cache.keys, cache.values, att, ctx.tables[cache.group], ctx.q_start, ctx.ctx_len,
                     ctx.seq_of_token, ctx.positions, nq, nkv, d, cache.page_size, s.scale,
                     s.window, ctx.max_q_len, ctx.max_ctx_len, ctx.min_q_len, ctx.seq_rows, **extra)
         if gate is not None:
             k.sigmoid_gate(att, gate)
-        return k.linear(att, self.o_proj, residual, residual=None if overwrite else residual, defer=True)
+        return self._output(att, residual, overwrite, hold)
+
+    def _output(self, att, residual, overwrite, hold):
+        """The output product, left pending or not even started."""
+        if hold:
+            return HeldProduct(att, self.o_proj)
+        return self.runtime.kernels.linear(att, self.o_proj, residual, residual=None if overwrite else residual,
+                                           defer=True)
 
     def _heads_from_the_product(self, x, ctx, cache, fused) -> bool:
         """Many rows on kernels that can do it: the q | k | v product normalises and

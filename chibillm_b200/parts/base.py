@@ -135,6 +135,15 @@ class PositionEncoding(Part):
         raise NotImplementedError
 
 
+@dataclass
+class HeldProduct:
+    """A sublayer's last product, x @ w^T, that has not been started (``hold=True``): a block whose
+    sublayers read the same input starts both of theirs together."""
+
+    x: torch.Tensor
+    w: torch.Tensor
+
+
 class Mixer(Part):
     """Mixes information between the tokens of a sequence.
 
@@ -155,6 +164,10 @@ class Mixer(Part):
     # is written over it instead of added to it (or is left pending).
     can_overwrite = False
 
+    # True: ``forward`` takes ``hold=True``, which says that the part's last product is to be left to the
+    # block: nothing is added to ``residual``, and a HeldProduct is returned.
+    can_hold = False
+
     def cache_need(self):
         return None
 
@@ -168,6 +181,7 @@ class FeedForward(Part):
 
     accepts_scaled_rows = False      # as for a mixer
     can_overwrite = False            # as for a mixer
+    can_hold = False                 # as for a mixer
     # a 32-bit vector that belongs to the result and that ``forward`` with ``overwrite=True`` leaves for the
     # block to add (None: there is none)
     output_bias = None

@@ -18,7 +18,11 @@ optional per-layer token input (parts/token_input.py).  The branches add into a
 32-bit array of their own; one kernel at the layer's end adds it to the residual
 with the scale, applies the token input and, when the next block's norm asks for
 it, writes that norm's output too (the block leaves that kernel pending, as a
-product is left pending by the other arrangement).
+product is left pending by the other arrangement).  Without a scale and a token
+input nothing comes between the branches and the residual: the branches then add
+into the residual itself, their last products are started together
+(``linear_pair``: for few rows the partial sums of both lie in one array that the
+next norm's kernel adds up in one go) and the block leaves the last one pending.
 
 "postnorm": the sublayers read the residual itself and the norms sit on their
 outputs, residual += norm(mixer(residual)), then residual += norm(ff(residual)),
@@ -262,6 +266,11 @@ class ParallelBlock(Block):
         self.token_input = None if layer.token_input is None else TokenInput(layer.token_input, names, runtime)
         self._parts = tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward, self.token_input)
                             if p is not None)
+        # the branches add straight into the residual
+        self.direct = layer.residual_scale == 1.0 and self.token_input is None
+        readers = (self.mixer, self.feed_forward)
+        self.scaled_ok = self.direct and all(p is None or p.accepts_scaled_rows for p in readers)
+        self.hold = self.direct and all(p is not None and p.can_hold for p in readers)
 
     def expected_tensors(self) -> List[TensorSpec]:
         out: List[TensorSpec] = []
@@ -281,8 +290,18 @@ class ParallelBlock(Block):
         rt = self.runtime
         k = rt.kernels
         x = ctx.workspace.get("block.normed", tuple(residual.shape), rt.dtype)
-        normed = self.mixer_norm.forward_fused(residual, pending, x, False)
+        normed = self.mixer_norm.forward_fused(residual, pending, x, self.scaled_ok)
         normed = x if normed is None else normed
+        if self.hold:
+            a = self.mixer.forward(normed, residual, ctx, cache, hold=True)
+            b = self.feed_forward.forward(normed, residual, ctx, hold=True)
+            return k.linear_pair(a.x, a.w, b.x, b.w, residual)
+        if self.direct:
+            left = self.mixer.forward(normed, residual, ctx, cache)
+            if left is None or self.feed_forward is None:
+                return left if self.feed_forward is None else self.feed_forward.forward(normed, residual, ctx)
+            left.add_into(residual)       # before the feed-forward starts split products of its own
+            return self.feed_forward.forward(normed, residual, ctx)
         delta = ctx.workspace.get("block.delta", tuple(residual.shape), torch.float32)
         k.zero(delta)
         left = self.mixer.forward(normed, delta, ctx, cache)

@@ -1,9 +1,9 @@
 """Dense gated feed-forward (SwiGLU): residual += down(silu(gate(x)) * up(x))
 (src/tensor/functions.cc:220-253).  gate and up are stacked into one matrix so
-one product yields both (src/qwen/qwen_weights.cc:13-16).  With another gate
-activation (the tanh form of gelu) or with biases on the three products the
-gate | up product is followed by one kernel that adds the biases, activates
-and multiplies.
+one product yields both (src/qwen/qwen_weights.cc:13-16).  With the tanh form of gelu
+as the gate's activation the same kernels do the work; with another activation or with
+biases on the three products the gate | up product is followed by one kernel that adds
+the biases, activates and multiplies.
 
 "table_experts": small gated feed-forwards without biases, chosen per token
 from a table by the token's id; the output is the mean of the chosen experts'.
@@ -32,7 +32,7 @@ from typing import Dict, List
 
 import torch
 
-from .base import FeedForward, Runtime, TensorSpec, register_feed_forward
+from .base import FeedForward, HeldProduct, Runtime, TensorSpec, register_feed_forward
 
 
 class GatedMLP(FeedForward):
@@ -43,6 +43,8 @@ class GatedMLP(FeedForward):
             raise ValueError("gated_mlp: the clamped gate has a positive limit and no biases")
         self.spec = spec
         self.plain_swiglu = spec.activation == "silu" and not spec.biases
+        # gates that the products' own epilogue applies
+        self.fused_gate = spec.activation in ("silu", "gelu_tanh") and not spec.biases
         self.bias_gate_up: torch.Tensor = None
         self.bias_down: torch.Tensor = None
         self.names = names
@@ -70,7 +72,7 @@ class GatedMLP(FeedForward):
             self.bias_gate_up = torch.cat([tensors[self.names["gate_bias"]].to(gate.dtype),
                                            tensors[self.names["up_bias"]].to(gate.dtype)]).contiguous()
             self.bias_down = tensors[self.names["down_bias"]].float().contiguous()
-        interleave = getattr(self.runtime.kernels, "interleave_gate_up", None) if self.plain_swiglu else None
+        interleave = getattr(self.runtime.kernels, "interleave_gate_up", None) if self.fused_gate else None
         self.gate_up_interleaved = interleave(gate, up) if interleave is not None else None
         # one of the two layouts is kept: blocks of 64 gate rows and their 64 up rows for the kernel
         # that applies SwiGLU itself, else gate rows followed by up rows
@@ -86,11 +88,26 @@ class GatedMLP(FeedForward):
     def launch_key(self, ctx):
         return ()
 
-    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, overwrite: bool = False):
+    @property
+    def can_hold(self):
+        return not self.spec.biases
+
+    def _output(self, act, residual, overwrite, hold):
+        """The down product, left pending or not even started."""
+        if hold:
+            return HeldProduct(act, self.down)
+        return self.runtime.kernels.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, ctx, overwrite: bool = False, hold: bool = False):
         k = self.runtime.kernels
         T = x.shape[0]
         inter = self.spec.intermediate_size
         act = ctx.workspace.get("mlp.act", (T, inter), self.runtime.dtype)
+        kind = self.spec.activation
+        if self.gate_up_interleaved is not None:
+            if not k.linear_swiglu(x, self.gate_up_interleaved, act, **({} if kind == "silu" else {"kind": kind})):
+                raise RuntimeError("gated_mlp: the fused kernel refused a shape it was prepared for")
+            return self._output(act, residual, overwrite, hold)
         if not self.plain_swiglu:
             gate_up = ctx.workspace.get("mlp.gate_up", (T, 2 * inter), self.runtime.dtype)
             k.linear(x, self.gate_up, gate_up)
@@ -100,11 +117,7 @@ class GatedMLP(FeedForward):
                 k.gated_activation(gate_up, self.bias_gate_up, act, self.spec.activation)
             if self.bias_down is not None:
                 k.add_row_vector(residual, self.bias_down)
-            return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
-        if self.gate_up_interleaved is not None:
-            if not k.linear_swiglu(x, self.gate_up_interleaved, act):
-                raise RuntimeError("gated_mlp: the fused kernel refused a shape it was prepared for")
-            return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
+            return self._output(act, residual, overwrite, hold)
         split = getattr(k, "linear_partial", None)
         pending = split(x, self.gate_up) if split is not None else None
         if pending is not None:
@@ -113,7 +126,7 @@ class GatedMLP(FeedForward):
             gate_up = ctx.workspace.get("mlp.gate_up", (T, 2 * inter), self.runtime.dtype)
             k.linear(x, self.gate_up, gate_up)
             k.swiglu(gate_up, act)
-        return k.linear(act, self.down, residual, residual=None if overwrite else residual, defer=True)
+        return self._output(act, residual, overwrite, hold)
 
 
 class DenseMLP(FeedForward):

@@ -48,6 +48,10 @@ class ReferenceKernels:
             y = residual + y
         out.copy_(y.to(out.dtype))
 
+    def linear_pair(self, x1, w1, x2, w2, residual):
+        self._count("linear_pair")
+        residual.add_(x1.float() @ w1.float().t() + x2.float() @ w2.float().t())
+
     def qk_norm_rope_append(self, qkv, q_out, k_cache, v_cache, q_norm_w, k_norm_w, inv_freq,
                             rotary_dim, eps, norm_offset, positions, seq_of_token, block_table,
                             nq, nkv, d, page_size, seq_rows=None):
@@ -385,7 +389,8 @@ class ReferenceKernels:
             acc.add_(wb * b.view_as(acc))
 
     def heads_prepare_append(self, proj, q_out, k_cache, v_cache, bias, q_norm, k_norm, eps, inv_freq, rotary_dim,
-                             positions, seq_of_token, block_table, nq, nk, nv, d, dv, page_size, seq_rows=None):
+                             positions, seq_of_token, block_table, nq, nk, nv, d, dv, page_size, seq_rows=None,
+                             unit_norm_eps=None, temperature=None):
         self._count("heads_prepare_append")
         T = proj.shape[0]
         append = k_cache is not None
@@ -398,6 +403,8 @@ class ReferenceKernels:
         def finish(x, w):
             if w is not None:
                 x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * w.float()
+            if unit_norm_eps is not None:
+                x = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + unit_norm_eps)
             if rotary_dim:
                 half = rotary_dim // 2
                 ang = pos[:, None] * inv_freq[:half].float()[None, :]
@@ -406,7 +413,11 @@ class ReferenceKernels:
                 x = torch.cat([u * c - v * s_, v * c + u * s_, x[..., rotary_dim:]], -1)
             return x
 
-        q_out.copy_(finish(row[:, :nq * d].reshape(T, nq, d), q_norm).reshape(T, nq * d).to(q_out.dtype))
+        q = finish(row[:, :nq * d].reshape(T, nq, d), q_norm)
+        if temperature is not None:
+            c, every = temperature
+            q = q * (1.0 + c * torch.log((positions.long() + 1).div(every, rounding_mode="floor").float() + 1.0))[:, None, None]
+        q_out.copy_(q.reshape(T, nq * d).to(q_out.dtype))
         if append:
             k = finish(row[:, nq * d:nq * d + nk * d].reshape(T, nk, d), k_norm)
             v = row[:, nq * d + nk * d:].reshape(T, nv, dv)
@@ -417,6 +428,39 @@ class ReferenceKernels:
             slots = (positions % page_size).long()
             k_cache[pages, :, slots, :] = k.to(k_cache.dtype)
             v_cache[pages, :, slots, :] = v.to(v_cache.dtype)
+
+    def latent_heads_append(self, proj, q_out, k_cache, kv_norm, eps, inv_freq, heads, kv_rank, rot, gates, positions,
+                            seq_of_token, block_table, page_size, seq_rows=None):
+        self._count("latent_heads_append")
+        p = proj.float()
+        T, kd = p.shape[0], rot + kv_rank
+        q = self._rotate_front(p[:, :heads * kd].reshape(T, heads, kd), positions, inv_freq, rot)
+        q_out.copy_(q.reshape(T, heads * kd).to(q_out.dtype))
+        at = heads * kd
+        if k_cache is not None:
+            c = p[:, at:at + kv_rank]
+            c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * kv_norm.float()
+            shared = self._rotate_front(p[:, at + kv_rank:at + kd], positions, inv_freq, rot)
+            pos = positions.long()
+            rows = seq_of_token.long() if seq_rows is None else seq_rows.long()[seq_of_token.long()]
+            pages = block_table[rows, pos // page_size].long()
+            assert (pages >= 0).all() and (pages < k_cache.shape[0]).all(), "append outside the pool"
+            k_cache[pages, 0, pos % page_size, :] = torch.cat([shared, c], dim=-1).to(k_cache.dtype)
+            at += kd
+        if gates is not None:
+            gates.copy_(torch.sigmoid(p[:, at:at + heads]))
+
+    def head_gate(self, x, gates, heads):
+        self._count("head_gate")
+        T = x.shape[0]
+        x.copy_((x.float().view(T, heads, -1) * gates[:, :, None]).view(x.shape).to(x.dtype))
+
+    def position_rows(self, x, factor, table, positions, weight, eps):
+        self._count("position_rows")
+        y = factor * x + table[positions.long()].float()
+        if weight is not None:
+            y = y * torch.rsqrt((y * y).mean(-1, keepdim=True) + eps) * weight.float()
+        x.copy_(y)
 
     def differential_combine(self, att, gate, lam, eps, out_scale, out, heads, dv, group):
         self._count("differential_combine")
