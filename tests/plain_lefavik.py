@@ -22,7 +22,7 @@ def gelu_tanh(z):
 
 def embed(ids, config, w):
     """The token's row times a constant, plus the position's row, normalised."""
-    x = w["embed"][ids] * config["embedding"]["scale"] + w["pos"][: len(ids)]
+    x = w["embed"][ids] * config.get("embedding", {}).get("scale", 1.0) + w["pos"][: len(ids)]
     return unit_rms(x, config["norm"]["eps"]) * w["embed.norm"]
 
 
@@ -71,7 +71,7 @@ def latent_rows(h, m, w, p, eps):
 
 
 def latent_attention(h, m, w, p, rows):
-    T, H, d, r, e = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
+    T, H, d, r, e = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m.get("vdim", m["dim"])
     latent, turned = rows
     q = (h @ w[p + "q"].T).view(T, H, d + r)
     q_turned = rotate_neighbours(q[..., d:], m["rot"]["base"], m["rot"]["dims"])
