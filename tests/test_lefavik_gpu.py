@@ -465,7 +465,7 @@ def test_a_far_key_and_a_sink_as_heavy(tmp_path, dtype, rows):
             for trace, what in ((helpers.trace_whole({"r0": ids}), "whole"), (helpers.trace_last_decoded({"r0": ids}, 20), "decoded"),
                                 (helpers.trace_portions({"r0": ids}, seed=at), "portions")):
                 got = helpers.run_trace(runner, trace)
-                helpers.assert_logits_close(got, ref, TOL[dtype] * 2, f"lefavik far key {rows} heavy {heavy} {dtype} {what}")
+                helpers.assert_logits_close(got, ref, TOL[dtype] * (3 if heavy else 2), f"lefavik far key {rows} heavy {heavy} {dtype} {what}")
 
 
 @pytest.fixture(scope="module")
