@@ -24,6 +24,7 @@
 #define CHIBI_UNIT_ID 7
 #include "common.cuh"
 #include "sm100.cuh"
+#include "attention_tc.cuh"
 #include "tensor_map.cuh"
 
 #ifndef CHIBI_HEAD_DIM
@@ -48,78 +49,11 @@ constexpr int NUM_BARS = 16;
 constexpr size_t ATC_SMEM = SMEM_TILES + NUM_BARS * 8 + 16 + 1024;
 constexpr uint32_t TMEM_S0 = 0, TMEM_S1 = 128, TMEM_O = 256;
 
-struct AttnTcParams {
-    const __nv_bfloat16* q;
-    __nv_bfloat16* out;
-    const int* block_table;
-    int table_stride;
-    const int* seq_rows;
-    const int* q_start;
-    const int* ctx_len;
-    int nq, nkv, group;
-    int page_size;
-    long long cache_rows;        // pages * nkv * page_size: rows of the [rows, D] view of a cache
-    int num_pages;
-    float scale_log2;
-    int window;
-    int chunk;                     // 0: none; else a row sees only keys of its own block of this many positions
-    int skip_single;
-    int* error;
-    // Options of the score (the kernel with one query tile per CTA only): a soft cap c replaces a
-    // scaled score s by c * tanh(s / c); a bias by distance then takes r1 * ln(1 + r2 * (pos - key))
-    // off, with r1 and r2 per query head.
-    float scale;                   // the plain scale
-    float softcap;                 // 0: none
-    const float* bias_r1;          // [nq] or null
-    const float* bias_r2;
-    // The kernel with one query tile per CTA may cut the keys of a row tile into kv_splits ranges,
-    // one CTA each (few query rows over a long context would leave most SMs idle otherwise): every
-    // CTA then leaves its unnormalised output, maximum and sum per row, and
-    // attn_prefill_merge_kernel puts the ranges together.
-    int kv_splits;                 // 1: none
-    float* part_o;                 // [tokens][nq][kv_splits][D]
-    float* part_ml;                // [tokens][nq][kv_splits][2]
-    const float* sink;             // [nq] or null: exp(sink[head]) joins the softmax's denominator, once
-};
+// Options of the score, compiled in: 0 none; 1 any of them (a soft cap, a bias of either kind); 2 a bias linear in
+// the distance and nothing else, which costs a multiply-add or two a score.
+constexpr int OPT_NONE = 0, OPT_ANY = 1, OPT_LINEAR = 2;
 
-// What the sink adds to a row's sum of weights, which is kept relative to the running maximum
-// `m` (in units of log2; -inf while no key has been seen, then the sum is relative to 0).
-__device__ __forceinline__ float sink_weight(const float* sink, int head, float m)
-{
-    return sink ? exp2f(sink[head] * 1.4426950408889634f - (m == -INFINITY ? 0.f : m)) : 0.f;
-}
-
-// Byte offset of element (row, col) of a [rows][64] bf16 tile laid out with the
-// 128-byte swizzle (what TMA writes and tcgen05.mma reads): 16-byte chunk c of
-// row r sits at chunk position c ^ (r % 8).
-__device__ __forceinline__ uint32_t swizzled_chunk(int row, int chunk)
-{
-    return (uint32_t)row * 128u + (uint32_t)((chunk ^ (row & 7)) << 4);
-}
-
-__device__ __forceinline__ float fast_exp2(float x)
-{
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
-// MN-major operand (here V: [key][d], d contiguous) in the same swizzled tiles:
-// leading byte offset = distance between the 64-wide slices of d, stride byte
-// offset = 8 keys * 128 B.
-__device__ __forceinline__ uint64_t make_mnmajor_sw128_desc(uint32_t smem_byte_addr, uint32_t lbo_bytes)
-{
-    uint64_t d = 0;
-    d |= static_cast<uint64_t>((smem_byte_addr & 0x3ffff) >> 4);
-    d |= static_cast<uint64_t>((lbo_bytes >> 4) & 0x3fff) << 16;
-    d |= static_cast<uint64_t>(1024 >> 4) << 32;
-    d |= static_cast<uint64_t>(1) << 46;
-    d |= static_cast<uint64_t>(2) << 61;
-    return d;
-}
-
-// OPT: the instantiation with the options of the score; the plain one is compiled without them.
-template <bool OPT>
+template <int OPT>
 __global__ void __launch_bounds__(ATC_THREADS)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        const AttnTcParams p)
@@ -318,8 +252,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const uint32_t lane_addr = tmem_base + (static_cast<uint32_t>(quarter * 32) << 16);
         // with options the scores are brought to their final form (in units of log2) right after
         // they are read, and the scale below is 1
-        constexpr bool options = OPT;
-        const float sl2 = options ? 1.f : p.scale_log2;
+        constexpr bool options = OPT == OPT_ANY;
+        const float sl2 = OPT != OPT_NONE ? 1.f : p.scale_log2;
         const int bias_head = kv_head * p.group + (live ? r - tok * p.group : 0);
         const float r1 = p.bias_r1 ? p.bias_r1[bias_head] : 0.f, r2 = p.bias_r2 ? p.bias_r2[bias_head] : 0.f;
         const bool linear_bias = p.bias_r1 && !p.bias_r2;       // r1 * distance instead of r1 * ln(1 + r2 * distance)
@@ -353,6 +287,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                     v -= linear_bias ? r1 * (float)(dist > 0 ? dist : 0) : r1 * __logf(1.f + r2 * (float)(dist > 0 ? dist : 0));
                     sv[i] = __float_as_uint(v * 1.4426950408889634f);
                 }
+            } else if (OPT == OPT_LINEAR) {
+                // score - slope * (pos - key), in units of log2; keys after pos are masked below
+                const float slope = r1 * 1.4426950408889634f, at0 = slope * (float)(key0 - pos);
+#pragma unroll
+                for (int i = 0; i < KEYS; ++i)
+                    sv[i] = __float_as_uint(fmaf(__uint_as_float(sv[i]), p.scale_log2, fmaf((float)i, slope, at0)));
             }
             // masks only where a row's visible range ends inside the tile; the warp takes one path
             const bool masked = __any_sync(0xffffffffu, key0 + KEYS - 1 > pos || key0 < first);
@@ -492,49 +432,6 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     }
 }
 
-// Puts the key ranges of attn_prefill_tc_kernel together: one block of D threads for each
-// (head, token of a sequence); ranges in order, eight at a time.
-__global__ void attn_prefill_merge_kernel(const AttnTcParams p)
-{
-    pdl_trigger();
-    const int seq = blockIdx.z, head = blockIdx.x, c = threadIdx.x;
-    const int t0 = p.q_start[seq];
-    const int q_len = p.q_start[seq + 1] - t0;
-    if ((int)blockIdx.y >= q_len || (q_len == 1 && p.skip_single))
-        return;
-    pdl_wait();
-    const size_t slot0 = ((size_t)(t0 + blockIdx.y) * p.nq + head) * p.kv_splits;
-    float m_run = -INFINITY, acc = 0.f, lsum = 0.f;
-    for (int s0 = 0; s0 < p.kv_splits; s0 += 8) {
-        float mv[8], lv[8], ov[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const bool in = s0 + u < p.kv_splits;
-            mv[u] = in ? p.part_ml[(slot0 + s0 + u) * 2] : -INFINITY;
-            lv[u] = in ? p.part_ml[(slot0 + s0 + u) * 2 + 1] : 0.f;
-            ov[u] = in ? p.part_o[(slot0 + s0 + u) * D + c] : 0.f;
-        }
-        float m_new = m_run;
-#pragma unroll
-        for (int u = 0; u < 8; ++u)
-            m_new = fmaxf(m_new, mv[u]);
-        const float base = m_new == -INFINITY ? 0.f : m_new;
-        const float keep = exp2f(m_run - base);       // 0 while nothing has been seen
-        acc *= keep;
-        lsum *= keep;
-#pragma unroll
-        for (int u = 0; u < 8; ++u) {
-            const float f = exp2f(mv[u] - base);
-            acc += ov[u] * f;
-            lsum += lv[u] * f;
-        }
-        m_run = m_new;
-    }
-    lsum += sink_weight(p.sink, head, m_run);
-    p.out[((size_t)(t0 + blockIdx.y) * p.nq + head) * D + c] = __float2bfloat16_rn(lsum > 0.f ? acc / lsum : 0.f);
-}
-
-
 // O[row, :] *= f for this thread's row of an output accumulator in TMEM (a rare
 // event: kept out of line so that its registers do not count against the loop).
 __device__ __noinline__ void rescale_output_row(uint32_t o_addr, float f)
@@ -569,7 +466,7 @@ constexpr int SMEM2_TILES = 2 * Q_BYTES + 4 * KV_TILE_BYTES;
 constexpr int NUM_BARS2 = 14;
 constexpr size_t ATC2_SMEM = SMEM2_TILES + NUM_BARS2 * 8 + 16 + 1024;
 
-template <bool OPT>
+template <int OPT>
 __global__ void __launch_bounds__(ATC2_THREADS, 1)
 attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const AttnTcParams p)
@@ -778,8 +675,8 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         float m = -INFINITY, l = 0.f;
         // options of the score: both passes over the row bring their piece to its final form (in
         // units of log2) right after it is read, and the scale below is 1
-        constexpr bool options = OPT;
-        const float sl2 = options ? 1.f : p.scale_log2;
+        constexpr bool options = OPT == OPT_ANY;
+        const float sl2 = OPT != OPT_NONE ? 1.f : p.scale_log2;
         const int bias_head = kv_head * p.group + (live ? r - tok * p.group : 0);
         const float r1 = p.bias_r1 ? p.bias_r1[bias_head] : 0.f, r2 = p.bias_r2 ? p.bias_r2[bias_head] : 0.f;
         const bool linear_bias = p.bias_r1 && !p.bias_r2;       // r1 * distance instead of r1 * ln(1 + r2 * distance)
@@ -796,9 +693,18 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             const bool masked = __any_sync(0xffffffffu, key0 + KEYS - 1 > pos || key0 < first);
             // With options the first pass brings a piece to its final form and writes it back to its
             // columns; the second pass reads finished (and masked) scores and changes nothing.
-            auto mask_piece = [&](uint32_t (&v)[32], int c0, bool second = false) {
+            // With a linear bias alone both passes make the scores anew; the second takes the exponents' base off
+            // on the way.
+            const float slope = OPT == OPT_LINEAR ? r1 * 1.4426950408889634f : 0.f;
+            const float at0 = OPT == OPT_LINEAR ? slope * (float)(key0 - pos) : 0.f;
+            auto mask_piece = [&](uint32_t (&v)[32], int c0, bool second = false, float off = 0.f) {
                 if (options && second)
                     return;
+                if (OPT == OPT_LINEAR) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i)
+                        v[i] = __float_as_uint(fmaf(__uint_as_float(v[i]), p.scale_log2, fmaf((float)(c0 + i), slope, at0 - off)));
+                }
                 if (options) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
@@ -862,12 +768,13 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             const float base = m == -INFINITY ? 0.f : m;
             float sum4[4] = { 0.f, 0.f, 0.f, 0.f };
             auto exp_piece = [&](uint32_t (&v)[32], int c0) {
-                mask_piece(v, c0, true);
+                mask_piece(v, c0, true, base);
                 uint32_t packed[16];
 #pragma unroll
                 for (int i = 0; i < 16; ++i) {
-                    const float p0 = fast_exp2(fmaf(__uint_as_float(v[2 * i]), sl2, -base));
-                    const float p1 = fast_exp2(fmaf(__uint_as_float(v[2 * i + 1]), sl2, -base));
+                    const float a = __uint_as_float(v[2 * i]), b = __uint_as_float(v[2 * i + 1]);
+                    const float p0 = fast_exp2(OPT == OPT_LINEAR ? a : fmaf(a, sl2, -base));
+                    const float p1 = fast_exp2(OPT == OPT_LINEAR ? b : fmaf(b, sl2, -base));
                     sum4[i & 3] += p0 + p1;
                     const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
                     packed[i] = *reinterpret_cast<const uint32_t*>(&h);
@@ -993,20 +900,25 @@ CHIBI_API int chibi_attention_prefill_tc(const void* q, const void* k_cache, con
     p.bias_r1 = bias_r1;
     p.bias_r2 = bias_r2;
     p.sink = sink;
-    const bool with_options = softcap > 0.f || bias_r1 != nullptr;
+    const int options = softcap > 0.f || bias_r2 ? OPT_ANY : (bias_r1 ? OPT_LINEAR : OPT_NONE);
     CUtensorMap mk, mv;
     if (!tensor_map_2d(k_cache, p.cache_rows, D, D, page_size, &mk)
         || !tensor_map_2d(v_cache, p.cache_rows, D, D, page_size, &mv))
         return CHIBI_ERR_UNSUPPORTED;
+    using Kernel = void (*)(const CUtensorMap, const CUtensorMap, const AttnTcParams);
+    static const Kernel one_tile[3] = { attn_prefill_tc_kernel<OPT_NONE>, attn_prefill_tc_kernel<OPT_ANY>,
+                                        attn_prefill_tc_kernel<OPT_LINEAR> };
+    static const Kernel two_tiles[3] = { attn_prefill_tc2_kernel<OPT_NONE>, attn_prefill_tc2_kernel<OPT_ANY>,
+                                         attn_prefill_tc2_kernel<OPT_LINEAR> };
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                             (int)ATC_SMEM);
-        if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                     (int)ATC_SMEM);
-        if (e != cudaSuccess)
-            return (int)e;
+        for (int i = 0; i < 3; ++i) {
+            cudaError_t e = cudaFuncSetAttribute(one_tile[i], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ATC_SMEM);
+            if (e == cudaSuccess)
+                e = cudaFuncSetAttribute(two_tiles[i], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ATC2_SMEM);
+            if (e != cudaSuccess)
+                return (int)e;
+        }
         configured = true;
     }
     const long long rows = (long long)max_q_len * p.group;
@@ -1017,22 +929,8 @@ CHIBI_API int chibi_attention_prefill_tc(const void* q, const void* k_cache, con
     if (cudaGetDevice(&device) == cudaSuccess)
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, device);
     if (variant == 2 || (variant == 0 && ctas2 >= sms)) {
-        static bool configured2 = false;
-        if (!configured2) {
-            cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc2_kernel<false>,
-                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ATC2_SMEM);
-            if (e == cudaSuccess)
-                e = cudaFuncSetAttribute(attn_prefill_tc2_kernel<true>,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ATC2_SMEM);
-            if (e != cudaSuccess)
-                return (int)e;
-            configured2 = true;
-        }
         const dim3 grid2((unsigned)((rows + 2 * ROWS - 1) / (2 * ROWS)), nkv, seqs);
-        if (with_options)
-            launch(attn_prefill_tc2_kernel<true>, grid2, dim3(ATC2_THREADS), ATC2_SMEM, stream, mk, mv, p);
-        else
-            launch(attn_prefill_tc2_kernel<false>, grid2, dim3(ATC2_THREADS), ATC2_SMEM, stream, mk, mv, p);
+        launch(two_tiles[options], grid2, dim3(ATC2_THREADS), ATC2_SMEM, stream, mk, mv, p);
         return launch_status();
     }
     if (kv_splits > 1) {
@@ -1045,13 +943,10 @@ CHIBI_API int chibi_attention_prefill_tc(const void* q, const void* k_cache, con
         p.part_ml = scratch + (size_t)tokens * nq * kv_splits * D;
     }
     const dim3 grid((unsigned)((rows + ROWS - 1) / ROWS), nkv, seqs * p.kv_splits);
-    if (with_options)
-        launch(attn_prefill_tc_kernel<true>, grid, dim3(ATC_THREADS), ATC_SMEM, stream, mk, mv, p);
-    else
-        launch(attn_prefill_tc_kernel<false>, grid, dim3(ATC_THREADS), ATC_SMEM, stream, mk, mv, p);
+    launch(one_tile[options], grid, dim3(ATC_THREADS), ATC_SMEM, stream, mk, mv, p);
     int st = launch_status();
     if (st == CHIBI_OK && p.kv_splits > 1) {
-        launch(attn_prefill_merge_kernel, dim3(nq, max_q_len, seqs), dim3(D), 0, stream, p);
+        launch(attn_prefill_merge_kernel<D>, dim3(nq, max_q_len, seqs), dim3(D), 0, stream, p);
         st = launch_status();
     }
     return st;

@@ -35,10 +35,19 @@ LIBRARIES: Dict[str, List[str]] = {
     "chibi_attention_mma": ["attention_mma.cu"],
     # prompt attention on tcgen05, head sizes 64 and 128
     "chibi_attention_tc": ["attention_tcgen05.cu"],
+    # the same for caches whose values are their keys, rows of 144 to 256 numbers
+    "chibi_attention_tied": ["attention_tied_tcgen05.cu"],
 }
 TCGEN05_ATTENTION_HEAD_DIMS = (64, 128)
 # head sizes whose attention library build_all() makes ahead of time
 PREBUILT_HEAD_DIMS = (16, 32, 48, 64, 128)
+PREBUILT_TIED_DIMS = (192, 256)
+
+
+def tied_on_tcgen05(dim: int) -> bool:
+    """Whether prompt attention over a cache with rows of ``dim`` numbers whose values are its keys has a kernel
+    of its own."""
+    return dim % 16 == 0 and 128 < dim <= 256
 
 
 class BuildError(RuntimeError):
@@ -230,7 +239,12 @@ def attention_tc_library(head_dim: int, verbose: bool = True) -> str:
     return ensure_library("chibi_attention_tc", (f"CHIBI_HEAD_DIM={head_dim}",), verbose)
 
 
-def prepare(head_dims: Sequence[int] = (), bfloat16: bool = True, verbose: bool = True) -> None:
+def attention_tied_library(row_dim: int, verbose: bool = True) -> str:
+    return ensure_library("chibi_attention_tied", (f"CHIBI_HEAD_DIM={row_dim}",), verbose)
+
+
+def prepare(head_dims: Sequence[int] = (), bfloat16: bool = True, verbose: bool = True,
+            tied_dims: Sequence[int] = ()) -> None:
     """Builds side by side what a model with these head sizes will load and is not there yet: the
     kernel library, the host runtime and, for bfloat16, the attention libraries of each head size
     that the tensor-core kernels take.  Loading them one after the other, each built when first
@@ -246,6 +260,9 @@ def prepare(head_dims: Sequence[int] = (), bfloat16: bool = True, verbose: bool 
                 jobs.append(lambda d=d: attention_library(d, verbose))
             if d in TCGEN05_ATTENTION_HEAD_DIMS:
                 jobs.append(lambda d=d: attention_tc_library(d, verbose))
+        for d in sorted(set(int(d) for d in tied_dims)):
+            if tied_on_tcgen05(d):
+                jobs.append(lambda d=d: attention_tied_library(d, verbose))
     with ThreadPoolExecutor(max_workers=len(jobs)) as pool:
         for done in [pool.submit(job) for job in jobs]:
             done.result()
@@ -256,6 +273,7 @@ def build_all(verbose: bool = True) -> List[str]:
     with ThreadPoolExecutor(max_workers=4) as pool:
         out += list(pool.map(lambda d: attention_library(d, verbose), PREBUILT_HEAD_DIMS))
         out += list(pool.map(lambda d: attention_tc_library(d, verbose), TCGEN05_ATTENTION_HEAD_DIMS))
+        out += list(pool.map(lambda d: attention_tied_library(d, verbose), PREBUILT_TIED_DIMS))
     return out
 
 

@@ -54,19 +54,22 @@ def make_runtime(dtype, device="cuda:0", kernels=None, spec=None) -> Runtime:
             # on a library built for the pair of sizes and single tokens on the plain kernel)
             def mixers(m):
                 return [x for side in (m.left, m.right) for x in mixers(side)] if m.kind == "parallel_mixers" else [m]
-            head_dims = set()
+            head_dims, tied_dims = set(), set()
             for layer in spec.layers:
                 for m in mixers(layer.mixer):
                     if m.kind == "latent_attention":
                         head_dims.add(m.rope_dim + m.kv_rank)        # one key head whose rows are the values too
+                        tied_dims.add(m.rope_dim + m.kv_rank)
                     if m.kind != "attention":
                         continue
+                    if m.tied_values:
+                        tied_dims.add(m.head_dim)
                     dv = getattr(m, "value_dim", None) or m.head_dim
                     if dv != m.head_dim:
                         head_dims.add((m.head_dim, dv))
                     else:
                         head_dims.add(m.head_dim)
-            build.prepare(head_dims, bfloat16=parse_dtype(dtype) == torch.bfloat16)
+            build.prepare(head_dims, bfloat16=parse_dtype(dtype) == torch.bfloat16, tied_dims=tied_dims)
         kernels = CudaKernels(device)
     return Runtime(device=device, dtype=parse_dtype(dtype), kernels=kernels)
 

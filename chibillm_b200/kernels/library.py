@@ -107,6 +107,10 @@ _SIGNATURES = {
         "chibi_attention_tc_head_dim": [],
         "chibi_attention_prefill_tc": [P, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, I, I, I, I, P, L, L, F, P, P, P, P, P],
     },
+    "chibi_attention_tied": {
+        "chibi_attention_tied_head_dim": [],
+        "chibi_attention_prefill_tied": [P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, I, I, I, I, P, L, L, P, P, P],
+    },
     "chibi_attention_mma": {
         "chibi_attention_mma_head_dim": [],
         "chibi_attention_mma_value_dim": [],

@@ -175,6 +175,7 @@ class CudaKernels:
         self.supports_graphs = True     # every op is a plain launch on the current stream
         self._attention_libs = {}
         self._attention_tc_libs = {}
+        self._attention_tied_libs = {}
         self.use_tcgen05_attention = True
         self._partial_bufs = [None, None]
         self._partial_turn = 0
@@ -214,7 +215,7 @@ class CudaKernels:
         if self.profiler is None:
             self.profiler = LaunchProfiler()
             self.lib = ProfiledLibrary(self.lib, self.profiler)
-            for libs in (self._attention_libs, self._attention_tc_libs):
+            for libs in (self._attention_libs, self._attention_tc_libs, self._attention_tied_libs):
                 for d in list(libs):
                     libs[d] = ProfiledLibrary(libs[d], self.profiler)
             self.supports_graphs = False
@@ -976,6 +977,29 @@ class CudaKernels:
                     return
             elif status != -2:
                 _check(status, "attention (tcgen05)")
+        elif mode & 2 and self.use_tcgen05_attention and build.tied_on_tcgen05(d) and page_size in (8, 16, 32) \
+                and v_cache.data_ptr() == k_cache.data_ptr() and softcap == 0.0 and bias_r1 is None and scale > 0.0:
+            # the same where the values are the keys and a cache row is wider
+            tied = self._attention_tied_libs.get(d)
+            if tied is None:
+                tied = self._load("chibi_attention_tied", (f"CHIBI_HEAD_DIM={d}",))
+                if tied.chibi_attention_tied_head_dim() != d:
+                    raise KernelError(f"the tied attention library for rows of {d} was built for another size")
+                tied = self._attention_tied_libs[d] = self._profiled(tied)
+            kv_splits = self.prompt_attention_key_ranges(seqs, nq, nkv, max_q_len, max_ctx_len)
+            part = self._scratch(q.shape[0] * nq * kv_splits * (d + 2)) if kv_splits > 1 else None
+            status = tied.chibi_attention_prefill_tied(
+                _ptr(q), _ptr(k_cache), _ptr(out), _ptr(block_table), block_table.stride(0), _ptr(seq_rows), _ptr(q_start),
+                _ptr(ctx_len), seqs, nq, nkv, page_size, k_cache.shape[0], float(scale), int(window or 0), int(chunk),
+                1 if mode & 1 else 0, int(max_q_len), kv_splits, _ptr(part), part.numel() if part is not None else 0,
+                q.shape[0], _ptr(sink), _ptr(self.error), self._stream())
+            if status == 0:
+                self.launches += 2 if kv_splits > 1 else 1
+                mode &= 1
+                if mode == 0:
+                    return
+            elif status != -2:
+                _check(status, "attention (tcgen05, tied values)")
         splits, scratch = 1, None
         if mode & 1:
             splits = self.decode_attention_splits(seqs, nq, nkv, max_ctx_len)

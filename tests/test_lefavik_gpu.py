@@ -354,6 +354,64 @@ def test_queries_cache_rows_and_gates(kernels, dtype, H, c, r):
     kernels.check_error_word()
 
 
+@pytest.mark.parametrize("d,H,page", [(144, 3, 8), (160, 2, 32), (192, 8, 16), (208, 5, 16), (224, 1, 8), (256, 32, 16), (256, 6, 32),
+                                      (192, 12, 64)])
+@pytest.mark.parametrize("window", [None, 100, 1])
+def test_prompt_attention_over_rows_that_are_keys_and_values(kernels, d, H, page, window):
+    """Several sequences in one step -- a whole prompt, a portion after a long context, two tokens, one token, a
+    prompt that fills its last page -- with pages of NaN around what was written; on the kernel for wide rows, and
+    (page of 64, or switched off) on the one that it stands for.  A short portion alone after a long context
+    runs in key ranges."""
+    g = torch.Generator().manual_seed(d + H)
+    held = [(0, 300), (1000, 40), (37, 2), (500, 1), (0, 192)]
+    T = sum(n for _, n in held)
+    pages = sum((c + n + page - 1) // page for c, n in held) + 4
+    order = torch.randperm(pages, generator=g).tolist()
+    cache = torch.full((pages, 1, page, d), float("nan"), dtype=torch.bfloat16)
+    table = torch.full((len(held) + 1, 1200 // page + 2), -1, dtype=torch.int32)
+    q = torch.randn(T, H, d, generator=g).to(torch.bfloat16)
+    sink, scale = torch.randn(H, generator=g), 3.0 / math.sqrt(d)
+    ref, at, starts, seq_of, positions = [], 0, [0], [], []
+    for i, (c, n) in enumerate(held):
+        rows = torch.randn(c + n, d, generator=g).to(torch.bfloat16)
+        for b in range((c + n + page - 1) // page):
+            pg = order.pop()
+            table[i + 1, b] = pg
+            part = rows[b * page:(b + 1) * page]
+            cache[pg, 0, :part.shape[0]] = part
+        seen = plain.visible(c + n, window)[c:]
+        scores = torch.einsum("ihd,jd->hij", q[at:at + n].double(), rows.double()) * scale
+        ref.append(torch.stack([plain.weights_with_sink(scores[h], seen, sink[h].double()) @ rows.double() for h in range(H)], 1))
+        at += n
+        starts.append(at)
+        seq_of += [i] * n
+        positions += list(range(c, c + n))
+    ref = torch.cat(ref).reshape(T, H * d)
+    cache, table, qd = cache.to(DEV), table.to(DEV), q.reshape(T, H * d).to(DEV)
+    lens = [c + n for c, n in held]
+
+    def run(which, **how):
+        lo, hi = starts[which[0]], starts[which[-1] + 1]
+        out = torch.full((hi - lo, H * d), float("nan"), dtype=torch.bfloat16, device=DEV)
+        ns = [held[i][1] for i in which]
+        kernels.attention(qd[lo:hi].contiguous(), cache, cache, out, table, i32([starts[i] - lo for i in which] + [hi - lo]),
+                          i32([lens[i] for i in which]), i32([seq_of[t] - which[0] for t in range(lo, hi)]), i32(positions[lo:hi]),
+                          H, 1, d, page, scale, window, max(ns), max(lens[i] for i in which), min(ns),
+                          i32([i + 1 for i in which]), sink=sink.to(DEV), **how)
+        kernels.check_error_word()
+        return out, ref[lo:hi]
+
+    for which in ([0, 1, 2, 3, 4], [1], [2], [4], [0]):
+        got, want = run(which)
+        close(got, want, 2e-2, f"rows of {d}, {H} heads, window {window}, sequences {which}")
+    kernels.use_tcgen05_attention = False
+    try:
+        got, want = run([0, 1, 2, 3, 4])
+    finally:
+        kernels.use_tcgen05_attention = True
+    close(got, want, 2e-2, f"rows of {d} on the other kernel")
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("T,H,n", [(1, 3, 33), (8, 32, 256), (300, 4, 48), (2000, 8, 128), (7, 1, 700)])
 def test_head_gate(kernels, dtype, T, H, n):
