@@ -375,7 +375,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         if (n_tiles > 0)
             mbar_wait(&o_full[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, p.error, 30);
         tcgen05_fence_after();
-        const int head = kv_head * p.group + (r - tok * p.group);
+        const int head = kv_head * p.group + (live ? r - tok * p.group : 0);      // (rows past the end have none)
         if (p.kv_splits > 1) {
             // one of several key ranges: the row as it stands, with its maximum and sum
             const size_t slot = ((size_t)(t0 + tok) * p.nq + head) * p.kv_splits + split;
@@ -815,7 +815,7 @@ attn_prefill_tc2_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         if (my_tiles > 0) {
             mbar_wait(&o_done[q], (my_tiles - 1) & 1, p.error, 48);
             tcgen05_fence_after();
-            const int head = kv_head * p.group + (r - tok * p.group);
+            const int head = kv_head * p.group + (live ? r - tok * p.group : 0);      // (rows past the end have none)
             l += sink_weight(p.sink, head, m);
             const float inv = l > 0.f ? 1.f / l : 0.f;
             __nv_bfloat16* dst_row = p.out + ((size_t)(t0 + tok) * p.nq + head) * D;

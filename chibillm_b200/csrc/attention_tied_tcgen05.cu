@@ -303,7 +303,7 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
         if (n_tiles > 0)
             mbar_wait(&o_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, p.error, 28);
         tcgen05_fence_after();
-        const int head = kv_head * p.group + (r - tok * p.group);
+        const int head = kv_head * p.group + (live ? r - tok * p.group : 0);      // (rows past the end have none)
         const bool ranged = p.kv_splits > 1;
         const size_t slot = ((size_t)(t0 + tok) * p.nq + head) * p.kv_splits + split;
         float inv = 1.f;
