@@ -5,11 +5,15 @@
 // One CTA owns 128 query rows of one key head, (token, head of the group) pairs, and walks over the keys in tiles of
 // 96.  A tile is fetched once: it is the K-major operand of S = Q K^T and the MN-major operand of O += P K.
 //
-//   warp 0      loads key tiles with TMA, one box per cache page and 64-wide slice of a row, three tiles deep
-//               (columns past the row's end come as zeros);
+//   warp 0      loads key tiles with TMA, three tiles deep: one box brings eight keys with all whole 64-wide
+//               slices of their rows (one more the rest of a row, zeros past its end).  A tile lies in shared memory
+//               as [8 keys][slice], a swizzle atom each: with a box per page and slice, 2 KB each, the loader took
+//               2,200 cycles a tile of 48 KB, and everything waited for it;
 //   warp 1      issues the MMAs:  S(j + 1) into one of two TMEM buffers before  O += P(j) K(j);
-//   warps 2..5  softmax: thread r owns query row r.  P = exp2(S * scale - max) goes back into the first columns of
-//               its S buffer as packed bfloat16 and is the A operand from there, so it never leaves TMEM.
+//   warps 2..9  softmax: two threads, of warps w and w + 4, share query row r, half of a tile's keys each (one warp
+//               to a scheduler would wait for its own results most of the time).  They exchange their halves' maxima
+//               through shared memory; P = exp2(S * scale - max) goes back into the first columns of its S buffer
+//               as packed bfloat16 and is the A operand from there, so it never leaves TMEM.
 //
 // The output accumulates in TMEM over all tiles and is rescaled there only when a row's maximum has grown by more
 // than 2^8.  TMEM: S at columns 0 and 128, O from 256 on.  All waits are bounded.
@@ -34,20 +38,39 @@ constexpr int ROWS = 128;                      // query rows per CTA = UMMA M
 constexpr int KEYS = 96;                       // keys per tile
 constexpr int STAGES = 3;
 constexpr int SLICES = (D + 63) / 64;          // 64-wide (128-byte) slices of a row
-constexpr int THREADS = 192;
+constexpr int WHOLE = D / 64;                  // of which are whole
+constexpr int GROUPS = KEYS / 8;               // keys of a tile, eight by eight
+constexpr int GROUP_BYTES = SLICES * 1024;
+constexpr int THREADS = 320;
+constexpr int HALF = KEYS / 2;                 // keys of a tile per softmax thread
 constexpr int Q_BYTES = SLICES * ROWS * 128;
 constexpr int TILE_BYTES = SLICES * KEYS * 128;
 constexpr int SMEM_TILES = Q_BYTES + STAGES * TILE_BYTES;
 constexpr int NUM_BARS = 2 * STAGES + 6;
-constexpr size_t SMEM = SMEM_TILES + NUM_BARS * 8 + 16 + 1024;
+constexpr int EXCHANGE_BYTES = 2 * 2 * ROWS * 4;
+constexpr size_t SMEM = SMEM_TILES + EXCHANGE_BYTES + NUM_BARS * 8 + 16 + 1024;
 static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
 constexpr uint32_t TMEM_O = 256;
 
-// O[row, :] *= f for this thread's row (a rare event: out of line so that its registers do not count against the loop).
-__device__ __noinline__ void rescale_row(uint32_t o_addr, float f)
+// A 128-byte-swizzled operand: leading and stride byte offsets as the layout above has them (a key group of eight
+// is the stride of both products; the slices of a row are the leading offset where the row is the N dimension).
+__device__ __forceinline__ uint64_t sw128_desc(uint32_t smem_byte_addr, uint32_t lbo_bytes, uint32_t sbo_bytes)
+{
+    uint64_t d = 0;
+    d |= static_cast<uint64_t>((smem_byte_addr & 0x3ffff) >> 4);
+    d |= static_cast<uint64_t>(lbo_bytes == 1 ? 1 : (lbo_bytes >> 4) & 0x3fff) << 16;
+    d |= static_cast<uint64_t>(sbo_bytes >> 4) << 32;
+    d |= static_cast<uint64_t>(1) << 46;
+    d |= static_cast<uint64_t>(2) << 61;
+    return d;
+}
+
+// O[row, columns] *= f for this thread's half of its row's runs of 16 columns (a rare event: out of line so that its
+// registers do not count against the loop).
+__device__ __noinline__ void rescale_row(uint32_t o_addr, int half, float f)
 {
 #pragma unroll 1
-    for (int c0 = 0; c0 < D; c0 += 16) {
+    for (int c0 = 16 * half; c0 < D; c0 += 32) {
         uint32_t v[16];
         tmem_load_32x16(o_addr + c0, v);
         tmem_load_wait();
@@ -60,18 +83,20 @@ __device__ __noinline__ void rescale_row(uint32_t o_addr, float f)
 }
 
 __global__ void __launch_bounds__(THREADS, 1)
-attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcParams p)
+attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ CUtensorMap map_rest,
+                         const AttnTcParams p)
 {
     pdl_enter();
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* q_s = smem;
     uint8_t* k_s = q_s + Q_BYTES;                  // STAGES tiles
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SMEM_TILES);
+    float* exchange = reinterpret_cast<float*>(smem + SMEM_TILES);           // [2][half][row]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SMEM_TILES + EXCHANGE_BYTES);
     uint64_t* k_full = bars;                       // [STAGES] TMA
     uint64_t* k_empty = bars + STAGES;             // [STAGES] MMA commit: both products of the tile are done
     uint64_t* s_full = bars + 2 * STAGES;          // [2] MMA commit
-    uint64_t* p_full = s_full + 2;                 // [2] 128 threads
+    uint64_t* p_full = s_full + 2;                 // [2] 256 threads
     uint64_t* o_done = p_full + 2;                 // [2] MMA commit: O holds tile j
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NUM_BARS);
 
@@ -110,7 +135,7 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
         }
         for (int i = 0; i < 2; ++i) {
             mbar_init(&s_full[i], 1);
-            mbar_init(&p_full[i], 128);
+            mbar_init(&p_full[i], 256);
             mbar_init(&o_done[i], 1);
         }
         fence_barrier_init();
@@ -148,13 +173,13 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
     const uint32_t tmem_base = *tmem_slot;
 
     if (warp == 0) {
-        // Lane i brings page i of every tile (at most 12 pages: page_size >= 8), looked up one tile ahead.
+        // Lane i brings keys 8 i .. 8 i + 7 of every tile (of one page: pages are multiples of eight keys), their
+        // page looked up one tile ahead.
         if (lane == 0)
             tma_prefetch_descriptor(&map);
-        const int pages_per_tile = KEYS / p.page_size;
         auto first_row_of = [&](int j) -> long long {
-            const int key = key_begin + j * KEYS + lane * p.page_size;
-            if (lane >= pages_per_tile || key >= key_end)
+            const int key = key_begin + j * KEYS + lane * 8;
+            if (lane >= GROUPS || key >= key_end)
                 return p.cache_rows;      // past the context: read outside the array, zeros
             const int page = table[key / p.page_size];
             if (page < 0 || page >= p.num_pages) {
@@ -162,7 +187,7 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
                     atomicExch(p.error, 3);
                 return p.cache_rows;
             }
-            return ((long long)page * p.nkv + kv_head) * p.page_size;
+            return ((long long)page * p.nkv + kv_head) * p.page_size + key % p.page_size;
         };
         long long row = n_tiles > 0 ? first_row_of(0) : 0;
         for (int j = 0; j < n_tiles; ++j) {
@@ -175,9 +200,10 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
                 mbar_arrive_expect_tx(&k_full[st], TILE_BYTES);
             }
             __syncwarp();
-            if (lane < pages_per_tile) {
-                for (int h = 0; h < SLICES; ++h)
-                    tma_load_2d(dst + h * (KEYS * 128) + lane * p.page_size * 128, &map, &k_full[st], h * 64, (int)row);
+            if (lane < GROUPS) {
+                tma_load_3d(dst + lane * GROUP_BYTES, &map, &k_full[st], 0, (int)row, 0);
+                if (WHOLE < SLICES)
+                    tma_load_2d(dst + lane * GROUP_BYTES + WHOLE * 1024, &map_rest, &k_full[st], WHOLE * 64, (int)row);
             }
             row = row_next;
         }
@@ -195,7 +221,7 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
                 for (int ks = 0; ks < D / 16; ++ks)
                     tcgen05_mma_bf16(tmem_base + (j & 1) * 128,
                                      make_kmajor_sw128_desc(q_addr + (ks >> 2) * (ROWS * 128) + (ks & 3) * 32),
-                                     make_kmajor_sw128_desc(k_addr + (ks >> 2) * (KEYS * 128) + (ks & 3) * 32), idesc_qk,
+                                     sw128_desc(k_addr + (ks >> 2) * 1024 + (ks & 3) * 32, 1, GROUP_BYTES), idesc_qk,
                                      ks > 0 ? 1u : 0u);
                 tcgen05_commit(&s_full[j & 1]);
             };
@@ -212,14 +238,14 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
 #pragma unroll
                 for (int ks = 0; ks < KEYS / 16; ++ks)
                     tcgen05_mma_bf16_a_tmem(tmem_base + TMEM_O, tmem_base + (j & 1) * 128 + ks * 8,
-                                            make_mnmajor_sw128_desc(k_addr + ks * 16 * 128, KEYS * 128), idesc_pv,
+                                            sw128_desc(k_addr + ks * 2 * GROUP_BYTES, 1024, GROUP_BYTES), idesc_pv,
                                             (j > 0 || ks > 0) ? 1u : 0u);
                 tcgen05_commit(&o_done[j & 1]);
                 tcgen05_commit(&k_empty[st]);
             }
         }
     } else {
-        const int quarter = warp & 3;
+        const int quarter = warp & 3, half = warp >= 6 ? 1 : 0;
         const int row = quarter * 32 + lane;                 // this thread's query row = its TMEM lane
         const int r = row0 + row;
         const bool live = r < rows_total;
@@ -237,31 +263,38 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
             mbar_wait(&s_full[j & 1], (j >> 1) & 1, p.error, 26);
             tcgen05_fence_after();
             const uint32_t s_addr = lane_addr + (j & 1) * 128;
-            uint32_t sv[KEYS];
+            uint32_t sv[HALF];
 #pragma unroll
-            for (int c0 = 0; c0 < KEYS; c0 += 32)
-                tmem_load_32x32(s_addr + c0, *reinterpret_cast<uint32_t(*)[32]>(&sv[c0]));
+            for (int c0 = 0; c0 < HALF; c0 += 16)
+                tmem_load_32x16(s_addr + half * HALF + c0, *reinterpret_cast<uint32_t(*)[16]>(&sv[c0]));
             tmem_load_wait();
             // masks only where a row's visible range ends inside the tile; the warp takes one path
             if (__any_sync(0xffffffffu, key0 + KEYS - 1 > pos || key0 < first)) {
 #pragma unroll
-                for (int i = 0; i < KEYS; ++i) {
-                    const int key = key0 + i;
+                for (int i = 0; i < HALF; ++i) {
+                    const int key = key0 + half * HALF + i;
                     if (!(key <= pos && key >= first))
                         sv[i] = 0xff800000u;                 // -inf
                 }
             }
             float mx4[4] = { -INFINITY, -INFINITY, -INFINITY, -INFINITY };
 #pragma unroll
-            for (int i = 0; i < KEYS; ++i)
+            for (int i = 0; i < HALF; ++i)
                 mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[i]));
-            const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * sl2;      // the scale is positive
+            float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * sl2;      // the scale is positive
+            // the other half's maximum; behind this barrier both halves of S are in registers, so P may overwrite it
+            float* slots = exchange + (j & 1) * 2 * ROWS;
+            slots[half * ROWS + row] = mx;
+            tcgen05_fence_before();
+            asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory");
+            tcgen05_fence_after();
+            mx = fmaxf(mx, slots[(half ^ 1) * ROWS + row]);
             const bool grow = mx > m + 8.f;                  // also true for the first visible key (m = -inf)
             if (__any_sync(0xffffffffu, grow && m != -INFINITY && j > 0)) {
                 // rescale what has accumulated: the product of tile j-1 must have landed first
                 mbar_wait(&o_done[(j - 1) & 1], ((j - 1) >> 1) & 1, p.error, 27);
                 tcgen05_fence_after();
-                rescale_row(o_addr, (grow && m != -INFINITY) ? fast_exp2(m - mx) : 1.f);
+                rescale_row(o_addr, half, (grow && m != -INFINITY) ? fast_exp2(m - mx) : 1.f);
             }
             if (grow) {
                 l *= (m == -INFINITY) ? 0.f : fast_exp2(m - mx);
@@ -270,17 +303,17 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
             const float base = m == -INFINITY ? 0.f : m;
             float sum4[4] = { 0.f, 0.f, 0.f, 0.f };
 #pragma unroll
-            for (int c0 = 0; c0 < KEYS; c0 += 32) {
-                uint32_t packed[16];
+            for (int c0 = 0; c0 < HALF; c0 += 16) {
+                uint32_t packed[8];
 #pragma unroll
-                for (int i = 0; i < 16; ++i) {
+                for (int i = 0; i < 8; ++i) {
                     const float p0 = fast_exp2(fmaf(__uint_as_float(sv[c0 + 2 * i]), sl2, -base));
                     const float p1 = fast_exp2(fmaf(__uint_as_float(sv[c0 + 2 * i + 1]), sl2, -base));
                     sum4[i & 3] += p0 + p1;
                     const __nv_bfloat162 h = __floats2bfloat162_rn(p0, p1);
                     packed[i] = *reinterpret_cast<const uint32_t*>(&h);
                 }
-                tmem_store_32x16(s_addr + (c0 >> 1), packed);
+                tmem_store_32x8(s_addr + ((half * HALF + c0) >> 1), packed);
             }
             l += (sum4[0] + sum4[1]) + (sum4[2] + sum4[3]);
             // rows past the context may hold anything (a page is loaded whole): make them zero, so that
@@ -288,9 +321,9 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
             if (key0 + KEYS > key_end) {
                 mbar_wait(&k_full[j % STAGES], (j / STAGES) & 1, p.error, 29);
                 uint8_t* tile = k_s + (j % STAGES) * TILE_BYTES;
-                for (int c = row; c < (key0 + KEYS - key_end) * (SLICES * 8); c += 128) {
+                for (int c = half * 128 + row; c < (key0 + KEYS - key_end) * (SLICES * 8); c += 256) {
                     const int krow = key_end - key0 + c / (SLICES * 8), chunk = c % (SLICES * 8);
-                    *reinterpret_cast<uint4*>(tile + (chunk >> 3) * (KEYS * 128) + swizzled_chunk(krow, chunk & 7)) =
+                    *reinterpret_cast<uint4*>(tile + (krow >> 3) * GROUP_BYTES + (chunk >> 3) * 1024 + swizzled_chunk(krow & 7, chunk & 7)) =
                         make_uint4(0, 0, 0, 0);
                 }
                 fence_proxy_async();
@@ -299,7 +332,12 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
             tcgen05_fence_before();
             mbar_arrive(&p_full[j & 1]);
         }
-        // the last product has landed: normalise and write the rows out
+        // the two halves' sums (the exponents' base is the same)
+        float* slots = exchange + (n_tiles & 1) * 2 * ROWS;
+        slots[half * ROWS + row] = l;
+        asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory");
+        l += slots[(half ^ 1) * ROWS + row];
+        // the last product has landed: normalise and write the rows out, every other run of 16 columns
         if (n_tiles > 0)
             mbar_wait(&o_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, p.error, 28);
         tcgen05_fence_after();
@@ -310,14 +348,14 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const AttnTcPa
         if (!ranged) {
             l += sink_weight(p.sink, head, m);
             inv = l > 0.f ? 1.f / l : 0.f;
-        } else if (live) {
+        } else if (live && half == 0) {
             // one of several key ranges: the row as it stands, with its maximum and sum
             p.part_ml[slot * 2] = m;
             p.part_ml[slot * 2 + 1] = l;
         }
         __nv_bfloat16* dst_row = p.out + ((size_t)(t0 + tok) * p.nq + head) * D;
 #pragma unroll 1
-        for (int c0 = 0; c0 < D; c0 += 16) {
+        for (int c0 = 16 * half; c0 < D; c0 += 32) {
             uint32_t ov[16];
             if (n_tiles > 0) {
                 tmem_load_32x16(o_addr + c0, ov);
@@ -361,7 +399,7 @@ CHIBI_API int chibi_attention_tied_head_dim() { return D; }
 
 // Attention of the sequences that bring more than one token (all sequences when skip_single is 0); `cache`
 // [pages][nkv][page_size][D] holds the keys, which are the values.  CHIBI_ERR_UNSUPPORTED for page sizes it does not
-// take (8, 16 and 32 are taken: a tile of 96 keys is whole pages).
+// take (multiples of eight are taken).
 CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, void* out, const int* block_table,
                                            int table_stride, const int* seq_rows, const int* q_start, const int* ctx_len,
                                            int seqs, int nq, int nkv, int page_size, int num_pages, float scale, int window,
@@ -373,7 +411,7 @@ CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, voi
         return CHIBI_OK;
     if (nkv <= 0 || nq % nkv != 0 || window < 0 || chunk < 0 || !(scale > 0.f) || max_q_len <= 0 || kv_splits < 1)
         return CHIBI_ERR_ARGUMENT;
-    if ((page_size != 8 && page_size != 16 && page_size != 32) || (reinterpret_cast<uintptr_t>(cache) & 15)
+    if (page_size < 8 || page_size % 8 != 0 || (reinterpret_cast<uintptr_t>(cache) & 15)
         || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(out) & 15))
         return CHIBI_ERR_UNSUPPORTED;
     AttnTcParams p {};
@@ -404,8 +442,9 @@ CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, voi
         p.part_o = scratch;
         p.part_ml = scratch + (size_t)tokens * nq * kv_splits * D;
     }
-    CUtensorMap map;
-    if (p.cache_rows > 2147483647LL || !tensor_map_2d(cache, p.cache_rows, D, D, page_size, &map))
+    CUtensorMap map, rest;
+    if (p.cache_rows > 2147483647LL || !tensor_map_of_rows(cache, p.cache_rows, D, D, 8, WHOLE, &map)
+        || !tensor_map_2d(cache, p.cache_rows, D, D, 8, &rest))
         return CHIBI_ERR_UNSUPPORTED;
     static bool configured = false;
     if (!configured) {
@@ -417,7 +456,7 @@ CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, voi
     }
     const long long rows = (long long)max_q_len * p.group;
     launch(attn_prefill_tied_kernel, dim3((unsigned)((rows + ROWS - 1) / ROWS), nkv, seqs * kv_splits), dim3(THREADS), SMEM,
-           stream, map, p);
+           stream, map, rest, p);
     int st = launch_status();
     if (st == CHIBI_OK && kv_splits > 1) {
         launch(attn_prefill_merge_kernel<D>, dim3(nq, max_q_len, seqs), dim3(D), 0, stream, p);

@@ -977,7 +977,7 @@ class CudaKernels:
                     return
             elif status != -2:
                 _check(status, "attention (tcgen05)")
-        elif mode & 2 and self.use_tcgen05_attention and build.tied_on_tcgen05(d) and page_size in (8, 16, 32) \
+        elif mode & 2 and self.use_tcgen05_attention and build.tied_on_tcgen05(d) and page_size % 8 == 0 \
                 and v_cache.data_ptr() == k_cache.data_ptr() and softcap == 0.0 and bias_r1 is None and scale > 0.0:
             # the same where the values are the keys and a cache row is wider
             tied = self._attention_tied_libs.get(d)

@@ -355,12 +355,12 @@ def test_queries_cache_rows_and_gates(kernels, dtype, H, c, r):
 
 
 @pytest.mark.parametrize("d,H,page", [(144, 3, 8), (160, 2, 32), (192, 8, 16), (208, 5, 16), (224, 1, 8), (256, 32, 16), (256, 6, 32),
-                                      (192, 12, 64)])
+                                      (192, 12, 64), (256, 3, 128)])
 @pytest.mark.parametrize("window", [None, 100, 1])
 def test_prompt_attention_over_rows_that_are_keys_and_values(kernels, d, H, page, window):
     """Several sequences in one step -- a whole prompt, a portion after a long context, two tokens, one token, a
     prompt that fills its last page -- with pages of NaN around what was written; on the kernel for wide rows, and
-    (page of 64, or switched off) on the one that it stands for.  A short portion alone after a long context
+    (switched off) on the one that it stands for.  A short portion alone after a long context
     runs in key ranges."""
     g = torch.Generator().manual_seed(d + H)
     held = [(0, 300), (1000, 40), (37, 2), (500, 1), (0, 192)]
