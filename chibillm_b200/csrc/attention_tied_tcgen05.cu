@@ -15,7 +15,9 @@
 //               through shared memory; P = exp2(S * scale - max) goes back into the first columns of its S buffer
 //               as packed bfloat16 and is the A operand from there, so it never leaves TMEM.
 //
-// The output accumulates in TMEM over all tiles and is rescaled there only when a row's maximum has grown by more
+// With one key head the query rows of a CTA are neighbours in memory: they come by TMA, and a full tile of output rows
+// leaves by TMA from where they were (with loads and stores by the threads a CTA's start and end took as long as
+// eleven tiles).  The output accumulates in TMEM over all tiles and is rescaled there only when a row's maximum has grown by more
 // than 2^8.  TMEM: S at columns 0 and 128, O from 256 on.  All waits are bounded.
 #define CHIBI_UNIT attention_tied_tcgen05
 #define CHIBI_UNIT_ID 16
@@ -46,7 +48,7 @@ constexpr int HALF = KEYS / 2;                 // keys of a tile per softmax thr
 constexpr int Q_BYTES = SLICES * ROWS * 128;
 constexpr int TILE_BYTES = SLICES * KEYS * 128;
 constexpr int SMEM_TILES = Q_BYTES + STAGES * TILE_BYTES;
-constexpr int NUM_BARS = 2 * STAGES + 6;
+constexpr int NUM_BARS = 2 * STAGES + 7;
 constexpr int EXCHANGE_BYTES = 2 * 2 * ROWS * 4;
 constexpr size_t SMEM = SMEM_TILES + EXCHANGE_BYTES + NUM_BARS * 8 + 16 + 1024;
 static_assert(SMEM <= 227 * 1024, "shared memory of one CTA");
@@ -82,9 +84,13 @@ __device__ __noinline__ void rescale_row(uint32_t o_addr, int half, float f)
     tmem_store_wait();
 }
 
+// Maps of the rows of the cache (boxes of 8 rows), of q and of the output (boxes of 128): all whole slices, the rest.
+struct TiedMaps {
+    CUtensorMap cache, cache_rest, q, q_rest, out, out_rest;
+};
+
 __global__ void __launch_bounds__(THREADS, 1)
-attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ CUtensorMap map_rest,
-                         const AttnTcParams p)
+attn_prefill_tied_kernel(const __grid_constant__ TiedMaps maps, const AttnTcParams p)
 {
     pdl_enter();
     extern __shared__ uint8_t smem_raw[];
@@ -98,6 +104,7 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
     uint64_t* s_full = bars + 2 * STAGES;          // [2] MMA commit
     uint64_t* p_full = s_full + 2;                 // [2] 256 threads
     uint64_t* o_done = p_full + 2;                 // [2] MMA commit: O holds tile j
+    uint64_t* q_full = o_done + 2;                 // TMA (one key head)
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NUM_BARS);
 
     // the row tiles with the most keys start first, for all key heads
@@ -138,14 +145,17 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
             mbar_init(&p_full[i], 256);
             mbar_init(&o_done[i], 1);
         }
+        mbar_init(q_full, 1);
         fence_barrier_init();
     }
     if (warp == 1) {
         tmem_alloc(tmem_slot, 512);
         tmem_relinquish();
     }
-    // query rows -> shared memory in the swizzled K-major layout (all threads help), eight loads of a thread at a time
-    for (int c0 = threadIdx.x; c0 < ROWS * (D / 8); c0 += 8 * THREADS) {
+    // query rows -> shared memory in the swizzled K-major layout: by TMA below, or all threads help, eight loads of a
+    // thread at a time
+    const bool neighbours = p.nkv == 1;
+    for (int c0 = threadIdx.x; !neighbours && c0 < ROWS * (D / 8); c0 += 8 * THREADS) {
         uint4 v[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -175,8 +185,17 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
     if (warp == 0) {
         // Lane i brings keys 8 i .. 8 i + 7 of every tile (of one page: pages are multiples of eight keys), their
         // page looked up one tile ahead.
-        if (lane == 0)
-            tma_prefetch_descriptor(&map);
+        if (lane == 0) {
+            tma_prefetch_descriptor(&maps.cache);
+            if (neighbours) {
+                // (rows past the sequence's end are somebody else's or zeros; their results go nowhere)
+                mbar_arrive_expect_tx(q_full, Q_BYTES);
+                tma_load_3d(q_s, &maps.q, q_full, 0, t0 * p.nq + row0, 0);
+                if (WHOLE < SLICES)
+                    tma_load_2d(q_s + WHOLE * (ROWS * 128), &maps.q_rest, q_full, WHOLE * 64, t0 * p.nq + row0);
+            }
+        }
+        __syncwarp();
         auto first_row_of = [&](int j) -> long long {
             const int key = key_begin + j * KEYS + lane * 8;
             if (lane >= GROUPS || key >= key_end)
@@ -201,9 +220,9 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
             }
             __syncwarp();
             if (lane < GROUPS) {
-                tma_load_3d(dst + lane * GROUP_BYTES, &map, &k_full[st], 0, (int)row, 0);
+                tma_load_3d(dst + lane * GROUP_BYTES, &maps.cache, &k_full[st], 0, (int)row, 0);
                 if (WHOLE < SLICES)
-                    tma_load_2d(dst + lane * GROUP_BYTES + WHOLE * 1024, &map_rest, &k_full[st], WHOLE * 64, (int)row);
+                    tma_load_2d(dst + lane * GROUP_BYTES + WHOLE * 1024, &maps.cache_rest, &k_full[st], WHOLE * 64, (int)row);
             }
             row = row_next;
         }
@@ -225,6 +244,8 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
                                      ks > 0 ? 1u : 0u);
                 tcgen05_commit(&s_full[j & 1]);
             };
+            if (neighbours)
+                mbar_wait(q_full, 0, p.error, 23);       // (also with no tile: nothing may be on its way at the end)
             if (n_tiles > 0)
                 issue_qk(0);
             for (int j = 0; j < n_tiles; ++j) {
@@ -354,6 +375,9 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
             p.part_ml[slot * 2 + 1] = l;
         }
         __nv_bfloat16* dst_row = p.out + ((size_t)(t0 + tok) * p.nq + head) * D;
+        // a full tile of neighbouring rows: through shared memory, where the queries were (the last product that reads
+        // them, S of the last tile, is long done)
+        const bool staged = neighbours && !ranged && row0 + ROWS <= rows_total && n_tiles > 0;
 #pragma unroll 1
         for (int c0 = 16 * half; c0 < D; c0 += 32) {
             uint32_t ov[16];
@@ -379,7 +403,20 @@ attn_prefill_tied_kernel(const __grid_constant__ CUtensorMap map, const __grid_c
 #pragma unroll
                 for (int u = 0; u < 4; ++u)
                     h[u] = __floats2bfloat162_rn(__uint_as_float(ov[8 * c + 2 * u]) * inv, __uint_as_float(ov[8 * c + 2 * u + 1]) * inv);
-                reinterpret_cast<uint4*>(dst_row + c0)[c] = *reinterpret_cast<uint4*>(h);
+                const int chunk = (c0 >> 3) + c;
+                uint4* dst = staged ? reinterpret_cast<uint4*>(q_s + (chunk >> 3) * (ROWS * 128) + swizzled_chunk(row, chunk & 7))
+                                    : reinterpret_cast<uint4*>(dst_row + c0) + c;
+                *dst = *reinterpret_cast<uint4*>(h);
+            }
+        }
+        if (staged) {
+            fence_proxy_async();
+            asm volatile("bar.sync 5, 256;" ::: "memory");
+            if (threadIdx.x == 64) {
+                tma_store_3d(&maps.out, q_s, 0, t0 * p.nq + row0, 0);
+                if (WHOLE < SLICES)
+                    tma_store_2d(&maps.out_rest, q_s + WHOLE * (ROWS * 128), WHOLE * 64, t0 * p.nq + row0);
+                tma_store_done();
             }
         }
     }
@@ -442,9 +479,14 @@ CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, voi
         p.part_o = scratch;
         p.part_ml = scratch + (size_t)tokens * nq * kv_splits * D;
     }
-    CUtensorMap map, rest;
-    if (p.cache_rows > 2147483647LL || !tensor_map_of_rows(cache, p.cache_rows, D, D, 8, WHOLE, &map)
-        || !tensor_map_2d(cache, p.cache_rows, D, D, 8, &rest))
+    TiedMaps maps;
+    const long long q_rows = tokens * nq;
+    if (p.cache_rows > 2147483647LL || q_rows <= 0 || q_rows > 2147483647LL
+        || !tensor_map_of_rows(cache, p.cache_rows, D, D, 8, WHOLE, &maps.cache)
+        || !tensor_map_2d(cache, p.cache_rows, D, D, 8, &maps.cache_rest)
+        || !tensor_map_of_rows(q, q_rows, D, D, ROWS, WHOLE, &maps.q) || !tensor_map_2d(q, q_rows, D, D, ROWS, &maps.q_rest)
+        || !tensor_map_of_rows(out, q_rows, D, D, ROWS, WHOLE, &maps.out)
+        || !tensor_map_2d(out, q_rows, D, D, ROWS, &maps.out_rest))
         return CHIBI_ERR_UNSUPPORTED;
     static bool configured = false;
     if (!configured) {
@@ -456,7 +498,7 @@ CHIBI_API int chibi_attention_prefill_tied(const void* q, const void* cache, voi
     }
     const long long rows = (long long)max_q_len * p.group;
     launch(attn_prefill_tied_kernel, dim3((unsigned)((rows + ROWS - 1) / ROWS), nkv, seqs * kv_splits), dim3(THREADS), SMEM,
-           stream, map, rest, p);
+           stream, maps, p);
     int st = launch_status();
     if (st == CHIBI_OK && kv_splits > 1) {
         launch(attn_prefill_merge_kernel<D>, dim3(nq, max_q_len, seqs), dim3(D), 0, stream, p);
